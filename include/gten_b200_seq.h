@@ -27,9 +27,10 @@ extern "C" {
 enum { GTB_SEQ_BF16 = 0, GTB_SEQ_F32 = 1 };                       /* compute mode */
 enum { GTB_MIX_SIGMOID_ATTN = 1, GTB_MIX_RETENTION = 2, GTB_MIX_MINGRU = 3, GTB_MIX_SOFTMAX_ATTN = 4, GTB_MIX_LATENT_ATTN = 5 };   /* branch kinds of a token mixer */
 enum { GTB_BLOCK_PARALLEL = 0, GTB_BLOCK_POSTNORM = 1, GTB_BLOCK_PRENORM = 2, GTB_BLOCK_SANDWICH = 3 };   /* layer styles */
-enum { GTB_FF_GEGLU = 0, GTB_FF_POLYNORM = 1, GTB_FF_EXPERTS = 2, GTB_FF_GATED_EXPERTS = 3, GTB_FF_SWIGLU = 4, GTB_FF_GROUP_EXPERTS = 5 };   /* feed-forward kinds */
-enum { GTB_NORM_RMS = 0, GTB_NORM_DYT = 1, GTB_NORM_LAYER = 2 };          /* norm of a pre-norm / sandwich layer and of the model's output */
+enum { GTB_FF_GEGLU = 0, GTB_FF_POLYNORM = 1, GTB_FF_EXPERTS = 2, GTB_FF_GATED_EXPERTS = 3, GTB_FF_SWIGLU = 4, GTB_FF_GROUP_EXPERTS = 5, GTB_FF_GELU = 6 };   /* feed-forward kinds */
+enum { GTB_NORM_RMS = 0, GTB_NORM_DYT = 1, GTB_NORM_LAYER = 2, GTB_NORM_LAYER_NB = 3 };   /* norm of a pre-norm / sandwich layer and of the model's output (NB: no bias) */
 enum { GTB_ROT_HALVES = 0, GTB_ROT_INTERLEAVED = 1 };             /* which entries a rotary pair takes: (i, i + dims/2) or (2i, 2i + 1) */
+enum { GTB_ROT_SCALE_WAVES = 0, GTB_ROT_SCALE_YARN = 1 };         /* how rot_factor > 0 rescales the frequencies (see rot_scaling) */
 
 /* One branch of a token mixer.  Tensors of branch b of layer i are "l<i>.mix.<name>.{q,k,v,o,...}".
  *  GTB_MIX_SIGMOID_ATTN: causal attention over the slot's K/V cache, `heads` query heads sharing `kv_heads` key/value
@@ -55,9 +56,16 @@ enum { GTB_ROT_HALVES = 0, GTB_ROT_INTERLEAVED = 1 };             /* which entri
  *    rotated, are one key part shared by all heads.  Plain keys uk c and values uv c per head; score = scale (q_plain . k_plain +
  *    q_rot . k_rot).  q_rank > 0: q = uq (unit-RMS(dq h) * dq.norm) instead of q h.  Rotation on the first rot_dims (<= rope_dim)
  *    entries of the rotated part in rot_layout.  window, sink as for GTB_MIX_SOFTMAX_ATTN (no pooled blocks); gated 3: head a's output
- *    times logistic(g h)_a, g with one row per head.  The slot caches only c and the rotated key part ([kv_rank + rope_dim] per token).
+ *    times logistic(g h)_a, g with one row per head; gated 2: one logistic gate per output entry (g [heads * vdim][width]).  The slot
+ *    caches only c and the rotated key part ([kv_rank + rope_dim] per token).  kv_from >= 0: no dkv; latents and rotated key parts are
+ *    those of layer kv_from's cache (an earlier GTB_MIX_LATENT_ATTN layer with the same kv_rank, rope_dim and rotation) under this
+ *    layer's own uk and uv.  rot_scaling GTB_ROT_SCALE_YARN as below.
  *    Tensors q | dq, dq.norm, uq; dkv, dkv.norm, uk, uv, sink, g, o.
- *  In sandwich layers (GTB_BLOCK_SANDWICH) GTB_MIX_SOFTMAX_ATTN and GTB_MIX_RETENTION take further parameters:
+ *  Frequency scaling (rot_factor > 0) of both attention kinds, rot_scaling: GTB_ROT_SCALE_WAVES as described for GTB_MIX_SOFTMAX_ATTN;
+ *    GTB_ROT_SCALE_YARN: with at(turns) = dims ln(rot_original / (2 pi turns)) / (2 ln rot_base), a = max(floor(at(rot_high)), 0),
+ *    b = min(ceil(at(rot_low)), dims - 1) and r_i = clamp((i - a) / max(b - a, 0.001), 0, 1) pair i turns with f_i (r_i / rot_factor +
+ *    1 - r_i), and the rotated entries are multiplied by 0.1 ln(rot_factor) + 1.
+ *  In sandwich layers (GTB_BLOCK_SANDWICH) GTB_MIX_SOFTMAX_ATTN, GTB_MIX_LATENT_ATTN and GTB_MIX_RETENTION take further parameters:
  *    softmax attention -- qk_norm 3: ONE RMS norm over the whole q projection (and one over the whole k projection) with weights q.norm
  *    [heads * maps * dim], k.norm [kv_heads * maps * dim]; rot_divide > 0: every rotary frequency is divided by it; chunk > 0: position i
  *    sees j <= i only when floor(i / chunk) = floor(j / chunk); gated 3: one logistic gate per head (g [heads][width]); bias: q, k, v
@@ -66,6 +74,13 @@ enum { GTB_ROT_HALVES = 0, GTB_ROT_INTERLEAVED = 1 };             /* which entri
  *    the same values; with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff (tensors lq1, lk1, lq2, lk2 [dim]) the head's output is
  *    (a1 - lambda a2) scaled to unit RMS over its vdim entries (eps of the model) times (1 - diff), then gated.  The cache of a maps-2 layer
  *    holds both key parts; kv_from names a layer of the same style with the same kv_heads, maps, dim, vdim.
+ *    conv > 0: every channel of q and k passes a causal convolution of `conv` taps right behind its projection (bias included),
+ *    y_t = sum_j w[c][j] u_(t - conv + 1 + j) with zeros before the sequence (tensors q.conv [heads * dim][conv], k.conv
+ *    [kv_heads * dim][conv]; the last conv - 1 projected values per channel are part of the slot); not together with qk_norm, rotation or
+ *    maps 2.  v_from_k: the values are the keys as they enter the cache (no v tensor, vdim = dim, one cache for both; not with
+ *    maps 2).  keep_first > 0: tokens j < keep_first stay visible outside the window or chunk, at their true distance (not with pool).  slopes: 2^(-8 (h + 1) / heads) (i - j) is taken off head h's scores (not with pool).
+ *    sink 2: the sink's score is 0 for every head (no tensor): the denominator holds one more 1.  out_bias: the out projection adds the
+ *    vector o.b (single-branch layers, both attention kinds).
  *    retention -- act 1: q, k, v <- silu(q), silu(k), silu(v) before the recurrence; out_norm 2: the concatenated heads are scaled to
  *    unit RMS TOGETHER and multiplied by the weight `norm` [heads * vdim]; gated 2: times logistic(g h). */
 typedef struct {
@@ -92,6 +107,12 @@ typedef struct {
     int bias;                        /* 1: q, k, v projections have bias vectors */
     int act;                         /* retention: 1 = silu on q, k, v */
     float rot_divide;                /* > 0: rotary frequencies are divided by it */
+    int rot_scaling;                 /* GTB_ROT_SCALE_* */
+    int conv;                        /* taps of the convolution behind the q and k projections; 0: none */
+    int v_from_k;                    /* 1: the values are the keys */
+    int keep_first;                  /* first tokens of the sequence that stay visible whatever the window */
+    int slopes;                      /* 1: head-wise slope times the distance is taken off the scores */
+    int out_bias;                    /* 1: the out projection has a bias vector */
 } gtb_seq_branch;
 
 /* Tensors of layer i beyond its branches'.  Parallel blocks: "l<i>.norm1" (one gain), "l<i>.mlp.{gate,up,down}", "l<i>.canon{1,2}".
@@ -115,8 +136,8 @@ typedef struct {
                                       * rewritten at once from the old ones, x_t <- sum_s hc<q>.mix[s][t] x_s + hc<q>.out[t] y.  One branch
                                       * (GTB_MIX_LATENT_ATTN);
                                       * GTB_BLOCK_SANDWICH: x += norm1b(mixer(norm1(x))); x += norm2b(ff(norm2(x))), four norms of kind norm_kind
-                                      * (GTB_NORM_LAYER or GTB_NORM_RMS with a plain weight); one or two branches (GTB_MIX_SOFTMAX_ATTN,
-                                      * GTB_MIX_RETENTION), each weighted by its out_scale */
+                                      * (GTB_NORM_LAYER, GTB_NORM_LAYER_NB or GTB_NORM_RMS with a plain weight); one or two branches
+                                      * (GTB_MIX_SOFTMAX_ATTN, GTB_MIX_RETENTION), each weighted by its out_scale, or one GTB_MIX_LATENT_ATTN */
     int ff_kind;                     /* GTB_FF_GEGLU: down(gelu_tanh(gate h) * (up h)); GTB_FF_POLYNORM: down(a N(z) + b N(z^2) + c N(z^3) + e),
                                       * z = up h, N = unit RMS over the ff values, (a, b, c, e) = tensor mlp.act; GTB_FF_EXPERTS: router outputs
                                       * 0 .. experts-1 are experts e<i>.down(relu(e<i>.up h)^2), the `identity` outputs after them return h;
@@ -129,10 +150,12 @@ typedef struct {
                                       * route_groups equal groups of neighbours, a group ranks by the sum of its two largest s, only experts of the
                                       * route_keep best groups can be chosen; the `top` largest s among them are chosen (ties to the lower index) and
                                       * weighted with route_scale * s (not renormalised); shared_ff > 0: one more expert of the same form and that
-                                      * inner width runs for every row with weight 1 */
+                                      * inner width runs for every row with weight 1;
+                                      * GTB_FF_GELU: down(gelu(up h)), gelu(z) = z (1 + erf(z / sqrt 2)) / 2 (tensors mlp.up, mlp.down) */
     int experts, top, identity;
     int norm_kind;                   /* GTB_BLOCK_PRENORM: GTB_NORM_RMS (x / rms(x) * w) or GTB_NORM_DYT (tanh(alpha x) * w + b, no statistics);
-                                      * GTB_BLOCK_SANDWICH: GTB_NORM_RMS or GTB_NORM_LAYER ((x - mean) / sqrt(variance + eps) * w + b) */
+                                      * GTB_BLOCK_SANDWICH: GTB_NORM_RMS, GTB_NORM_LAYER ((x - mean) / sqrt(variance + eps) * w + b) or
+                                      * GTB_NORM_LAYER_NB (the same without b) */
     int shared_ff;
     int route_groups, route_keep;    /* GTB_FF_GROUP_EXPERTS (0 groups counts as 1, 0 kept as all) */
     float route_scale;
@@ -149,10 +172,12 @@ typedef struct {
     int max_rows;                    /* rows per pass over the weights (longer steps are cut into passes); 0: default */
     float embed_scale;               /* embedding rows are multiplied by this (0 counts as 1) */
     int final_norm;                  /* 0: one gain; 1: weight vector stored around zero (1 + w); 2: Dynamic Tanh, tensors final.norm, final.norm.alpha, final.norm.b;
-                                      * 3: layer norm, tensors final.norm, final.norm.b */
+                                      * 3: layer norm, tensors final.norm, final.norm.b; 4: layer norm without bias, tensor final.norm */
     int streams;                     /* pre-norm layers: copies of the residual stream under hyper-connections (all equal to the embedding output at
                                       * the start, summed at the end); 0: one stream, plain residual sum */
     float logit_softcap;             /* > 0: logits <- cap * tanh(logits / cap) */
+    float logit_scale;               /* logits are multiplied by this, before the cap (0 counts as 1) */
+    int tied_head;                   /* 1: the output matrix is the embedding table (without embed_scale); no tensor head */
 } gtb_seq_config;
 
 typedef struct gtb_seq_model* gtb_seq_t;

@@ -44,7 +44,7 @@ def needs_build(target: str = "llama") -> bool:
     if not lib.exists():
         return True
     t = lib.stat().st_mtime
-    deps = list(CSRC.glob("*.cu")) + list(CSRC.glob("*.cuh")) + list(CSRC.glob("*.h")) + [HERE.parent / "include" / "gten_b200.h"]
+    deps = list(CSRC.glob("*.cu")) + list(CSRC.glob("*.cuh")) + list(CSRC.glob("*.h")) + list((HERE.parent / "include").glob("gten_b200*.h"))
     return any(d.stat().st_mtime > t for d in deps)
 
 

@@ -54,12 +54,14 @@ struct TensorDest {
     int group = 0, group_stride = 0;   // matrix rows placed in groups of `group` rows, `group_stride` rows apart (0: contiguous)
     int split_cols = 0;                // > 0: columns placed in blocks of split_cols, block j at dst + j * split_stride elements
     size_t split_stride = 0;
+    void* also = nullptr;              // a second copy of the matrix, row stride also_ld (a tied output matrix)
+    int also_ld = 0;
     bool loaded = false;
 };
 
 struct BranchW {
     gtb_seq_branch d{};
-    std::vector<float> decay, inv_freq;
+    std::vector<float> decay, inv_freq, slopes;
     int q_off = 0, k_off = 0, v_off = 0, g_off = 0, a_off = 0;
     int kq = 0, kk = 0, kv = 0;   // projection widths
     float* d_pb = nullptr;
@@ -73,6 +75,9 @@ struct BranchW {
     // sandwich layers
     float* d_onorm = nullptr;                       // retention: weight of the norm over the concatenated heads
     float* d_lam[4] = {nullptr, nullptr, nullptr, nullptr};     // differential attention: lq1, lk1, lq2, lk2
+    float* d_slope = nullptr;                       // distance slopes [heads]
+    float* d_conv = nullptr;                        // weights of the convolution behind the projections [q channels | k channels][taps]
+    float rot_amp = 1.0f;                           // factor on cos and sin of the rotation
 };
 
 struct LayerW {
@@ -85,7 +90,8 @@ struct LayerW {
     float* d_gain = nullptr;
     bool gu_inter = false;     // gate and up rows interleaved in groups of 32 (what the fused tensor-core epilogue reads)
     // post-norm style
-    float *d_bias = nullptr;   // bias of the fused branch projection [n1] (minGRU), or null
+    float *d_bias = nullptr;   // bias of the fused branch projection [n1], or null
+    float *d_obias = nullptr;  // bias of the out projection [width], or null
     float *norm1 = nullptr, *norm2 = nullptr;
     bf16 *w_up = nullptr, *w_down = nullptr, *w_router = nullptr;
     float *d_act = nullptr, *d_corr = nullptr;
@@ -108,6 +114,8 @@ struct Run {
     void *kc[2] = {nullptr, nullptr}, *vc[2] = {nullptr, nullptr};
     float* state[2] = {nullptr, nullptr};
     float* tail = nullptr;
+    float* ctail = nullptr;                 // last taps - 1 projected values of the convolution behind the projections [n_slots][taps - 1][channels]
+    int ctail_n = 0;                        // floats per slot
     float *pk = nullptr, *pv = nullptr;     // mean key / value of every completed block of `pool` tokens [n_slots][max_blocks][kv_heads * dim|vdim]
     int max_blocks = 0;
 };
@@ -128,6 +136,8 @@ struct gtb_seq_model {
     // pre-norm style: copies of the stream, latent attention workspace, shared expert
     int ns = 1;                                  // copies of the stream
     bool prenorm = false, sandwich = false;
+    float* convQ = nullptr;                      // queries after the convolution behind their projection [max_rows][heads * dim]
+    int conv_q_max = 0;
     float* qk_sc = nullptr;                      // scales of the whole-projection q / k norm [max_rows][2]
     float *xs = nullptr, *hc_one = nullptr, *latQ = nullptr, *latQA = nullptr, *Y2 = nullptr, *shw = nullptr;
     void *opQ = nullptr, *opO = nullptr;
@@ -206,6 +216,44 @@ void want_vector(gtb_seq_model* m, const std::string& name, float* dst, int rows
 }
 
 size_t osz(const gtb_seq_model* m) { return m->cfg.mode == GTB_SEQ_F32 ? 4 : 2; }
+// Rotary frequencies of a branch (in double, rounded once) and the factor on cos and sin that goes with them: base^(-2k/dims), rescaled when
+// rot_factor > 0 -- by wavelength (long ones slowed down by rot_factor, a linear blend between two bounds), or by YaRN's ramp over the pair
+// index -- and divided by rot_divide
+void rot_table(const gtb_seq_branch& d, std::vector<float>& inv_freq, float& amp) {
+    inv_freq.resize(d.rot_dims / 2);
+    amp = 1.0f;
+    const double fac = d.rot_factor, orig = d.rot_original, n = d.rot_dims, base = d.rot_base;
+    const bool yarn = fac > 0.0 && d.rot_scaling == GTB_ROT_SCALE_YARN;
+    double a = 0.0, b = 0.0;
+    if (yarn) {
+        auto at = [&](double turns) { return n * log(orig / (2.0 * M_PI * turns)) / (2.0 * log(base)); };
+        a = std::max(floor(at(d.rot_high)), 0.0);
+        b = std::min(ceil(at(d.rot_low)), n - 1.0);
+        amp = (float)(0.1 * log(fac) + 1.0);
+    }
+    for (int k = 0; k < d.rot_dims / 2; k++) {
+        double f = pow(base, -2.0 * k / n);
+        if (yarn) {
+            const double r = std::min(1.0, std::max(0.0, (k - a) / std::max(b - a, 0.001)));
+            f = f / fac * r + f * (1.0 - r);
+        } else if (fac > 0.0) {
+            const double wl = 2.0 * M_PI / f, lo = d.rot_low, hi = d.rot_high;
+            if (wl > orig / lo) f = f / fac;
+            else if (!(wl < orig / hi)) { const double sm = (orig / wl - lo) / (hi - lo); f = (1.0 - sm) * f / fac + sm * f; }
+        }
+        if (d.rot_divide > 0.0f) f /= (double)d.rot_divide;
+        inv_freq[k] = (float)f;
+    }
+}
+int upload_rot_table(gtb_seq_model* m, BranchW& b) {
+    if (b.d.rot_dims <= 0) return GTB_OK;
+    rot_table(b.d, b.inv_freq, b.rot_amp);
+    int rc = dalloc_t(m, &b.d_inv_freq, b.inv_freq.size());
+    if (rc) return rc;
+    // (same stream as the allocation's zero fill: a copy on another stream could be overtaken by it)
+    GTB_CUDA(cudaMemcpyAsync(b.d_inv_freq, b.inv_freq.data(), b.inv_freq.size() * sizeof(float), cudaMemcpyHostToDevice, ctx().stream));
+    return GTB_OK;
+}
 // fp32 values of recurrent state one slot holds for a branch
 size_t state_floats(const gtb_seq_branch& d) { return d.kind == GTB_MIX_MINGRU ? (size_t)d.dim : (size_t)d.heads * d.dim * d.vdim; }
 constexpr int GRU_CHUNK = 32;               // rows per chunk of the chunked minGRU scan
@@ -334,6 +382,7 @@ SoftAttn soft_args(const gtb_seq_model* m, const BranchW& b, const Run& run) {
     a.q_off = b.q_off; a.k_off = b.k_off; a.v_off = b.v_off; a.g_off = b.g_off; a.a_off = b.a_off;
     a.own_kv = b.d.kv_from < 0; a.max_ctx = m->cfg.max_ctx; a.max_blocks = run.max_blocks;
     a.maps = b.d.maps > 1 ? b.d.maps : 1; a.chunk = b.d.chunk; a.out_scale = b.d.out_scale; a.qk_sc = m->qk_sc;
+    a.rot_amp = b.rot_amp; a.keep = b.d.keep_first; a.slope = b.d_slope; a.v_is_k = b.d.v_from_k;
     if (a.maps > 1) { a.gate = 0; a.out_scale = 1.0f; }       // the maps are combined, gated and weighted afterwards
     return a;
 }
@@ -514,7 +563,7 @@ int run_retention(gtb_seq_model* m, const PassTables& t, int R, int S, const Run
 // ---- sandwich layers ---------------------------------------------------------------------------------------------------------
 NormArgs sw_norm(const gtb_seq_model* m, const LayerW& l, int q) {          // q: 0 norm1, 1 norm1b, 2 norm2, 3 norm2b
     NormArgs n{};
-    n.kind = l.d.norm_kind; n.w = l.sn_w[q]; n.b = l.sn_b[q]; n.eps = m->cfg.eps;
+    n.kind = l.d.norm_kind == GTB_NORM_LAYER_NB ? GTB_NORM_LAYER : l.d.norm_kind; n.w = l.sn_w[q]; n.b = l.sn_b[q]; n.eps = m->cfg.eps;      // (no bias: sn_b is null)
     return n;
 }
 
@@ -528,6 +577,40 @@ void sandwich_add(int R, size_t smem, const float* Y, const float* Y2, const flo
     else k_sandwich_add<OT, 4><<<R, 256, smem, st>>>(Y, Y2, Yg, pair_dst, top, W, post, x, next, op, ld_op, rn);
 }
 
+// The convolution behind the q and k projections of a softmax-attention branch: convolved queries to m->convQ, keys (and plain values) to the
+// slots' caches, the slots' histories brought up to date.
+template <typename OT, int V>
+void launch_qk_conv(const PassTables& t, const ConvArgs& a, const float* P, int ldp, int R, int rows_per, float* tail, float* Q, OT* kc, OT* vc, int every_one) {
+    const dim3 grid((R + rows_per - 1) / rows_per, ((a.nq + a.nk + a.nv) / V + 127) / 128);
+    cudaStream_t st = ctx().stream;
+    switch (a.taps) {
+        case 1: k_qk_conv<OT, V, 1><<<grid, 128, 0, st>>>(t, a, P, ldp, R, rows_per, tail, Q, kc, vc, every_one); break;
+        case 2: k_qk_conv<OT, V, 2><<<grid, 128, 0, st>>>(t, a, P, ldp, R, rows_per, tail, Q, kc, vc, every_one); break;
+        case 3: k_qk_conv<OT, V, 3><<<grid, 128, 0, st>>>(t, a, P, ldp, R, rows_per, tail, Q, kc, vc, every_one); break;
+        case 4: k_qk_conv<OT, V, 4><<<grid, 128, 0, st>>>(t, a, P, ldp, R, rows_per, tail, Q, kc, vc, every_one); break;
+        default: k_qk_conv<OT, V, 0><<<grid, 128, 0, st>>>(t, a, P, ldp, R, rows_per, tail, Q, kc, vc, every_one); break;
+    }
+}
+template <typename OT>
+int run_qk_conv(gtb_seq_model* m, const PassTables& t, int R, int S, const Run& run, int bi, const LayerW& l) {
+    const BranchW& b = l.br[bi];
+    ConvArgs a{};
+    const bool own = b.d.kv_from < 0;
+    a.nq = b.kq; a.nk = own ? b.kk : 0; a.nv = own && !b.d.v_from_k ? b.kv : 0; a.off = b.q_off; a.taps = b.d.conv; a.w = b.d_conv;
+    a.max_ctx = m->cfg.max_ctx; a.k_ld = b.d.kv_heads * b.d.dim; a.v_ld = b.d.kv_heads * b.d.vdim;
+    const bool vec = ((a.nq | a.nk | a.nv | a.off | l.n1 | a.k_ld | a.v_ld) & 3) == 0;
+    const int rows_per = R >= 512 ? 16 : R >= 64 ? 4 : 1, every_one = R == S && a.taps <= 4;
+    if (vec) launch_qk_conv<OT, 4>(t, a, m->P, l.n1, R, rows_per, run.ctail, m->convQ, (OT*)run.kc[bi], (OT*)run.vc[bi], every_one);
+    else launch_qk_conv<OT, 1>(t, a, m->P, l.n1, R, rows_per, run.ctail, m->convQ, (OT*)run.kc[bi], (OT*)run.vc[bi], every_one);
+    GTB_LAUNCHED();
+    if (a.taps > 1 && !every_one) {
+        const int nc = a.nq + a.nk;
+        k_canon_tail<<<dim3(S, (nc + 255) / 256), 256, 0, ctx().stream>>>(t, m->P + a.off, l.n1, nc, a.taps, run.ctail);
+        GTB_LAUNCHED();
+    }
+    return GTB_OK;
+}
+
 // One softmax-attention branch of a sandwich layer on R rows: projections in m->P, output into the out-projection operand.
 template <typename OT>
 int run_soft_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const Run& run, int bi, const LayerW& l, bool portions, int n_qtiles) {
@@ -535,14 +618,23 @@ int run_soft_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const R
     const gtb_seq_config& c = m->cfg;
     const BranchW& b = l.br[bi];
     OT* opC = (OT*)m->opC;
-    const SoftAttn a = soft_args(m, b, run);
-    const int M = a.maps, units = a.heads * M, nk = a.own_kv ? a.kv_heads * M : 0;
+    SoftAttn a = soft_args(m, b, run);
+    const int M = a.maps, units = a.heads * M, nk = a.own_kv ? a.kv_heads * M : 0, nv = a.own_kv && !a.v_is_k ? a.kv_heads : 0;
+    const float* Q = m->P;                   // where the attention kernels read the queries
+    int ldq = l.n1;
     if (a.qk_norm == 3) {
         k_proj_rms<<<R, 256, 0, st>>>(m->P, l.n1, a.q_off, units * a.dim, a.k_off, nk * a.dim, c.eps, m->qk_sc);
         GTB_LAUNCHED();
     }
-    k_sattn_prep<OT><<<dim3(R, (units + nk + (a.own_kv ? a.kv_heads : 0) + 3) / 4), 128, 0, st>>>(t, a, m->P, l.n1, (OT*)run.kc[bi], (OT*)run.vc[bi]);
-    GTB_LAUNCHED();
+    if (b.d.conv > 0) {
+        int rc = run_qk_conv<OT>(m, t, R, S, run, bi, l);
+        if (rc) return rc;
+        Q = m->convQ; ldq = b.kq;
+        a.q_off = 0; a.gate_src = m->P; a.gate_ld = l.n1;
+    } else {
+        k_sattn_prep<OT><<<dim3(R, (units + nk + nv + 3) / 4), 128, 0, st>>>(t, a, m->P, l.n1, (OT*)run.kc[bi], (OT*)run.vc[bi]);
+        GTB_LAUNCHED();
+    }
     // two maps per head: the units' outputs stay fp32 (their difference is taken afterwards), unit-major in m->O
     float* of = M > 1 ? m->O : nullptr;
     const int ldf = units * a.vdim;
@@ -551,25 +643,26 @@ int run_soft_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const R
     const size_t smem = (a.dim + 128 + 33) * sizeof(float);
     int done = -1;
     if (portions && sizeof(OT) == 2 && a.dim <= 128 && a.vdim <= 128)
-        done = sattn_mma(t, a, S, n_qtiles, m->P, l.n1, (const bf16*)run.kc[bi], (const bf16*)run.vc[bi], nullptr, nullptr, (bf16*)opC, l.kout_p, of, ldf);
+        done = sattn_mma(t, a, S, n_qtiles, Q, ldq, (const bf16*)run.kc[bi], (const bf16*)run.vc[bi], nullptr, nullptr, (bf16*)opC, l.kout_p, of, ldf);
     if (done > 0) return done;
     if (done < 0 && !portions && R <= SPLIT_MAX_ROWS && m->sattn_part) {
         int max_keys = c.max_ctx;
         if (a.window > 0) max_keys = std::min(max_keys, a.window);
         if (a.chunk > 0) max_keys = std::min(max_keys, a.chunk);
+        max_keys = std::min(c.max_ctx, max_keys + a.keep);
         const int splits = std::max(1, std::min(32, (max_keys + 127) / 128));
         if (splits > 1) {
-            k_sattn_split<OT><<<dim3(R, units, splits), 128, smem, st>>>(t, a, m->P, l.n1, (const OT*)run.kc[bi], (const OT*)run.vc[bi], nullptr, nullptr, m->sattn_part, R);
+            k_sattn_split<OT><<<dim3(R, units, splits), 128, smem, st>>>(t, a, Q, ldq, (const OT*)run.kc[bi], (const OT*)run.vc[bi], nullptr, nullptr, m->sattn_part, R);
             GTB_LAUNCHED();
-            if (of) k_sattn_join<float><<<dim3(R, units), 128, 0, st>>>(af, m->P, l.n1, m->sattn_part, R, splits, of, ldf);
-            else k_sattn_join<OT><<<dim3(R, units), 128, 0, st>>>(a, m->P, l.n1, m->sattn_part, R, splits, opC, l.kout_p);
+            if (of) k_sattn_join<float><<<dim3(R, units), 128, 0, st>>>(af, Q, ldq, m->sattn_part, R, splits, of, ldf);
+            else k_sattn_join<OT><<<dim3(R, units), 128, 0, st>>>(a, Q, ldq, m->sattn_part, R, splits, opC, l.kout_p);
             GTB_LAUNCHED();
             done = 0;
         }
     }
     if (done < 0) {
-        if (of) k_sattn<OT, float><<<dim3(R, units), 128, smem, st>>>(t, af, m->P, l.n1, (const OT*)run.kc[bi], (const OT*)run.vc[bi], nullptr, nullptr, of, ldf);
-        else k_sattn<OT, OT><<<dim3(R, units), 128, smem, st>>>(t, a, m->P, l.n1, (const OT*)run.kc[bi], (const OT*)run.vc[bi], nullptr, nullptr, opC, l.kout_p);
+        if (of) k_sattn<OT, float><<<dim3(R, units), 128, smem, st>>>(t, af, Q, ldq, (const OT*)run.kc[bi], (const OT*)run.vc[bi], nullptr, nullptr, of, ldf);
+        else k_sattn<OT, OT><<<dim3(R, units), 128, smem, st>>>(t, a, Q, ldq, (const OT*)run.kc[bi], (const OT*)run.vc[bi], nullptr, nullptr, opC, l.kout_p);
         GTB_LAUNCHED();
     }
     if (of) {
@@ -583,11 +676,133 @@ int run_soft_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const R
     return GTB_OK;
 }
 
+// ---- latent attention (pre-norm and sandwich layers) ---------------------------------------------------------------------------
+LatAttn lat_args(const gtb_seq_model* m, const BranchW& b) {
+    LatAttn a{};
+    a.heads = b.d.heads; a.dim = b.d.dim; a.rope = b.d.rope_dim; a.vdim = b.d.vdim; a.rank = b.d.kv_rank; a.q_rank = b.d.q_rank;
+    a.rot_dims = b.d.rot_dims; a.rot_layout = b.d.rot_layout; a.inv_freq = b.d_inv_freq; a.kv_norm = b.d_kvnorm; a.q_norm = b.d_qnorm;
+    a.eps = m->cfg.eps; a.q_off = b.q_off; a.kv_off = b.kv_off; a.g_off = b.g_off; a.a_off = b.a_off; a.c_ld = b.c_ld; a.max_ctx = m->cfg.max_ctx;
+    a.rot_amp = b.rot_amp; a.own_kv = b.d.kv_from < 0;
+    return a;
+}
+// the absorbed form as a softmax attention with one K/V head over the latent cache: keys [latent | rotated part], values the latent
+SoftAttn lat_soft_args(const gtb_seq_model* m, const BranchW& b) {
+    SoftAttn a{};
+    a.heads = b.d.heads; a.kv_heads = 1; a.dim = b.d.kv_rank + b.d.rope_dim; a.vdim = b.d.kv_rank;
+    a.scale = b.d.scale; a.eps = m->cfg.eps; a.window = b.d.window; a.sink = b.d_sink;
+    a.k_ld = a.v_ld = b.c_ld; a.own_kv = 1; a.max_ctx = m->cfg.max_ctx;
+    return a;
+}
+
+template <int VPW>
+int launch_lat_dec_mma(const PassTables& t, const SoftAttn& a, int R, int splits, const float* QA, int ldqa, const bf16* cache, float* part) {
+    const int DP = (a.dim + 15) & ~15;
+    const size_t smem = (size_t)(16 + 64) * (DP + 8) * 2 + 16 * (64 + 8) * 2 + 64 * sizeof(float);
+    static size_t allowed = 48 * 1024;
+    if (smem > 200 * 1024) return -1;
+    if (smem > allowed) { GTB_CUDA(cudaFuncSetAttribute(k_lat_dec_mma<VPW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); allowed = smem; }
+    k_lat_dec_mma<VPW><<<dim3(R, (a.heads + 15) / 16, splits), 128, smem, ctx().stream>>>(t, a, QA, ldqa, cache, part, R);
+    GTB_LAUNCHED();
+    return GTB_OK;
+}
+// -1: sizes outside the kernel (the caller takes the row kernels)
+int lat_dec_mma(const PassTables& t, const SoftAttn& a, int R, int splits, const float* QA, int ldqa, const bf16* cache, float* part) {
+    if (a.vdim <= 128) return launch_lat_dec_mma<32>(t, a, R, splits, QA, ldqa, cache, part);
+    if (a.vdim <= 256) return launch_lat_dec_mma<64>(t, a, R, splits, QA, ldqa, cache, part);
+    if (a.vdim <= 512) return launch_lat_dec_mma<128>(t, a, R, splits, QA, ldqa, cache, part);
+    return -1;
+}
+
+// The latent-attention branch of a layer on R rows: projections in m->P, gated output into the out-projection operand.  Prompt portions in
+// bf16 mode expand keys and values of the visible range from the cached latents and run the tensor-core softmax attention; everything else
+// runs the absorbed form on the row kernels.
+template <typename OT>
+int run_latent_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const Run& run, const LayerW& l, bool portions, const int* seg_lens, const int* seg_slots,
+                      int n_qtiles) {
+    cudaStream_t st = ctx().stream;
+    const gtb_seq_config& c = m->cfg;
+    OT* opC = (OT*)m->opC;
+    const BranchW& b = l.br[0];
+    const bool expand = portions && sizeof(OT) == 2 && seg_slots && m->latKx && b.d.dim + b.d.rope_dim <= 128 && b.d.vdim <= 128;
+    const LatAttn a = lat_args(m, b);
+    const int hd = a.dim + a.rope, parts = (a.own_kv ? 1 : 0) + (a.q_rank > 0 ? 1 : 0);
+    int rc;
+    if (parts > 0) {
+        k_lat_prep<OT><<<dim3(R, parts), 128, 0, st>>>(t, a, m->P, l.n1, (OT*)run.kc[0], (OT*)m->opQ, b.qrank_p);
+        GTB_LAUNCHED();
+    }
+    const float* Q = m->P;
+    int ldq = l.n1, q0 = b.q_off;
+    if (a.q_rank > 0) {
+        ldq = a.heads * hd;
+        rc = product<OT>(m, m->opQ, b.qrank_p, b.w_uq, b.qrank_p, m->latQ, ldq, R, a.heads * hd, b.qrank_p, nullptr, 0);
+        if (rc) return rc;
+        Q = m->latQ; q0 = 0;
+    }
+    if (expand) {
+        const int ld_qr = a.heads * hd, nx = a.heads * (a.dim + a.vdim);
+        k_lat_qrot<<<R, 128, 0, st>>>(t, a, Q, ldq, q0, m->latQ, ld_qr);
+        GTB_LAUNCHED();
+        for (int s = 0; s < S; s++) {
+            const int slot = seg_slots[s], p0 = m->host_pos[slot];
+            const int lo = b.d.window > 0 ? std::max(0, p0 - b.d.window + 1) : 0, n = p0 + seg_lens[s] - lo;
+            const bf16* src = (const bf16*)run.kc[0] + ((size_t)slot * c.max_ctx + lo) * b.c_ld;
+            rc = product<OT>(m, src, b.c_ld, b.w_uk, b.rank_p, m->latX, nx, n, nx, b.rank_p, nullptr, 0);      // uk and uv rows are one matrix
+            if (rc) return rc;
+            k_lat_pack<<<n, 256, 0, st>>>(a, m->latX, n, slot, lo, (const bf16*)run.kc[0], m->latKx, m->latVx);
+            GTB_LAUNCHED();
+        }
+        SoftAttn sa{};
+        sa.heads = sa.kv_heads = a.heads; sa.dim = hd; sa.vdim = a.vdim; sa.scale = b.d.scale; sa.eps = c.eps; sa.window = b.d.window; sa.sink = b.d_sink;
+        sa.gate = b.d.gated; sa.q_off = 0; sa.gate_src = m->P; sa.gate_ld = l.n1; sa.g_off = b.g_off; sa.a_off = b.a_off; sa.own_kv = 1; sa.max_ctx = c.max_ctx;
+        rc = sattn_mma(t, sa, S, n_qtiles, m->latQ, ld_qr, m->latKx, m->latVx, nullptr, nullptr, (bf16*)opC, l.kout_p);
+        if (rc < 0) return gtb::fail(GTB_ERR_STATE, "head sizes outside the tiled attention kernel");
+        return rc;
+    }
+    k_lat_qabs<<<dim3(R, a.heads, (a.rank + 127) / 128), 128, (hd + 512) * sizeof(float), st>>>(t, a, Q, ldq, q0, b.w_uk, b.rank_p, m->latQA);
+    GTB_LAUNCHED();
+    const SoftAttn sa = lat_soft_args(m, b);
+    const int ldqa = a.heads * sa.dim, ld_ol = (a.heads * a.rank + 7) / 8 * 8;
+    const size_t smem = (sa.dim + 128 + 33) * sizeof(float);
+    bool done = false;
+    if (sizeof(OT) == 2 && m->fused_attn && !portions && R <= SPLIT_MAX_ROWS && m->sattn_part) {
+        // decode rows in bf16 mode: 16 heads per CTA on tensor cores, one CTA per 64 keys of the longest key list this layer can meet
+        const int max_keys = sa.window > 0 ? std::min(c.max_ctx, sa.window) : c.max_ctx;
+        const int splits = std::max(1, std::min(32, (max_keys + 63) / 64));
+        rc = lat_dec_mma(t, sa, R, splits, m->latQA, ldqa, (const bf16*)run.kc[0], m->sattn_part);
+        if (rc > 0) return rc;
+        if (rc == 0) {
+            k_sattn_join<OT><<<dim3(R, sa.heads), 128, 0, st>>>(sa, m->latQA, ldqa, m->sattn_part, R, splits, (OT*)m->opO, ld_ol);
+            GTB_LAUNCHED();
+            done = true;
+        }
+    }
+    if (!done && !portions && R <= SPLIT_MAX_ROWS && m->sattn_part) {
+        const int max_keys = sa.window > 0 ? std::min(c.max_ctx, sa.window) : c.max_ctx;
+        const int splits = std::max(1, std::min(32, (max_keys + 127) / 128));
+        if (splits > 1) {
+            k_sattn_split<OT><<<dim3(R, sa.heads, splits), 128, smem, st>>>(t, sa, m->latQA, ldqa, (const OT*)run.kc[0], (const OT*)run.kc[0], nullptr, nullptr, m->sattn_part, R);
+            GTB_LAUNCHED();
+            k_sattn_join<OT><<<dim3(R, sa.heads), 128, 0, st>>>(sa, m->latQA, ldqa, m->sattn_part, R, splits, (OT*)m->opO, ld_ol);
+            GTB_LAUNCHED();
+            done = true;
+        }
+    }
+    if (!done) {
+        k_sattn<OT><<<dim3(R, sa.heads), 128, smem, st>>>(t, sa, m->latQA, ldqa, (const OT*)run.kc[0], (const OT*)run.kc[0], nullptr, nullptr, (OT*)m->opO, ld_ol);
+        GTB_LAUNCHED();
+    }
+    const int n_out = a.heads * a.vdim;
+    k_lat_vup<OT><<<dim3(R, std::max(1, std::min(std::max(1, 4096 / R), (n_out + 7) / 8))), 256, 0, st>>>(a, (const OT*)m->opO, ld_ol, b.w_uv, b.rank_p, m->P, l.n1, b.d.gated, opC, l.kout_p);
+    GTB_LAUNCHED();
+    return GTB_OK;
+}
+
 // One layer of the sandwich style on R rows: x += norm1b(mixer(norm1(x))); x += norm2b(ff(norm2(x))).  opA holds norm1(x) on entry; on
 // return it holds `next` of the new stream (the following layer's norm1) when next.w is set.
 template <typename OT>
-int run_sandwich_layer(gtb_seq_model* m, const PassTables& t, int R, int S, const Run& run, const LayerW& l, bool portions, const int* seg_lens, int n_qtiles,
-                       const NormArgs& next) {
+int run_sandwich_layer(gtb_seq_model* m, const PassTables& t, int R, int S, const Run& run, const LayerW& l, bool portions, const int* seg_lens, const int* seg_slots,
+                       int n_qtiles, const NormArgs& next) {
     cudaStream_t st = ctx().stream;
     const gtb_seq_config& c = m->cfg;
     const int W = c.width, wp = m->wp;
@@ -596,10 +811,11 @@ int run_sandwich_layer(gtb_seq_model* m, const PassTables& t, int R, int S, cons
     if (rc) return rc;
     for (int bi = 0; bi < l.d.n_branches; bi++) {
         if (l.br[bi].d.kind == GTB_MIX_SOFTMAX_ATTN) rc = run_soft_branch<OT>(m, t, R, S, run, bi, l, portions, n_qtiles);
+        else if (l.br[bi].d.kind == GTB_MIX_LATENT_ATTN) rc = run_latent_branch<OT>(m, t, R, S, run, l, portions, seg_lens, seg_slots, n_qtiles);
         else rc = run_retention<OT>(m, t, R, S, run, bi, l, portions, seg_lens);
         if (rc) return rc;
     }
-    rc = product<OT>(m, opC, l.kout_p, l.w_out, l.kout_p, m->Y, W, R, W, l.kout_p, nullptr, 0);
+    rc = product<OT>(m, opC, l.kout_p, l.w_out, l.kout_p, m->Y, W, R, W, l.kout_p, l.d_obias, 0);
     if (rc) return rc;
     // few rows and a routed feed-forward next: the residual update also computes the router's logits from the operand row it has just formed
     // and picks the experts (two launches less per layer on a decode step)
@@ -614,6 +830,25 @@ int run_sandwich_layer(gtb_seq_model* m, const PassTables& t, int R, int S, cons
     sandwich_add<OT>(R, rn.w ? rn_smem : 0, m->Y, nullptr, nullptr, nullptr, 0, W, sw_norm(m, l, 1), m->x, l.ff > 0 ? sw_norm(m, l, 2) : next, opA, wp, rn);
     GTB_LAUNCHED();
     if (l.ff == 0) return GTB_OK;
+    if (l.d.ff_kind == GTB_FF_GELU) {
+        bool act_done = false;
+        if (sizeof(OT) == 2 && m->use_tensor && m->gp && R >= m->tensor_min_rows) {
+            rc = seq_gemm_bf16_gelu(m->gp, opA, wp, l.w_up, wp, opC, l.kfp, R, l.ff, wp);
+            if (rc > 0) return rc;
+            if (rc == 0) { ctx().launches++; act_done = true; }
+        }
+        if (!act_done) {
+            rc = product<OT>(m, opA, wp, l.w_up, wp, m->G, l.ff, R, l.ff, wp, nullptr, 0);
+            if (rc) return rc;
+            k_gelu_rows<OT><<<dim3(R, std::max(1, std::min((l.kfp + 255) / 256, std::max(1, 2048 / R)))), 256, 0, st>>>(m->G, l.ff, opC, l.kfp);
+            GTB_LAUNCHED();
+        }
+        rc = product<OT>(m, opC, l.kfp, l.w_down, l.kfp, m->Y, W, R, W, l.kfp, nullptr, 0);
+        if (rc) return rc;
+        sandwich_add<OT>(R, 0, m->Y, nullptr, nullptr, nullptr, 0, W, sw_norm(m, l, 3), m->x, next, opA, wp, GroupRouteNext{});
+        GTB_LAUNCHED();
+        return GTB_OK;
+    }
     if (l.d.ff_kind == GTB_FF_SWIGLU) {
         bool act_done = false;
         if (sizeof(OT) == 2 && m->use_tensor && m->gp && R >= m->tensor_min_rows && l.gu_inter) {
@@ -697,41 +932,6 @@ int hc_boundary(gtb_seq_model* m, int R, PendingUpdate& pend, const float* hc_ne
     return GTB_OK;
 }
 
-LatAttn lat_args(const gtb_seq_model* m, const BranchW& b) {
-    LatAttn a{};
-    a.heads = b.d.heads; a.dim = b.d.dim; a.rope = b.d.rope_dim; a.vdim = b.d.vdim; a.rank = b.d.kv_rank; a.q_rank = b.d.q_rank;
-    a.rot_dims = b.d.rot_dims; a.rot_layout = b.d.rot_layout; a.inv_freq = b.d_inv_freq; a.kv_norm = b.d_kvnorm; a.q_norm = b.d_qnorm;
-    a.eps = m->cfg.eps; a.q_off = b.q_off; a.kv_off = b.kv_off; a.g_off = b.g_off; a.a_off = b.a_off; a.c_ld = b.c_ld; a.max_ctx = m->cfg.max_ctx;
-    return a;
-}
-// the absorbed form as a softmax attention with one K/V head over the latent cache: keys [latent | rotated part], values the latent
-SoftAttn lat_soft_args(const gtb_seq_model* m, const BranchW& b) {
-    SoftAttn a{};
-    a.heads = b.d.heads; a.kv_heads = 1; a.dim = b.d.kv_rank + b.d.rope_dim; a.vdim = b.d.kv_rank;
-    a.scale = b.d.scale; a.eps = m->cfg.eps; a.window = b.d.window; a.sink = b.d_sink;
-    a.k_ld = a.v_ld = b.c_ld; a.own_kv = 1; a.max_ctx = m->cfg.max_ctx;
-    return a;
-}
-
-template <int VPW>
-int launch_lat_dec_mma(const PassTables& t, const SoftAttn& a, int R, int splits, const float* QA, int ldqa, const bf16* cache, float* part) {
-    const int DP = (a.dim + 15) & ~15;
-    const size_t smem = (size_t)(16 + 64) * (DP + 8) * 2 + 16 * (64 + 8) * 2 + 64 * sizeof(float);
-    static size_t allowed = 48 * 1024;
-    if (smem > 200 * 1024) return -1;
-    if (smem > allowed) { GTB_CUDA(cudaFuncSetAttribute(k_lat_dec_mma<VPW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); allowed = smem; }
-    k_lat_dec_mma<VPW><<<dim3(R, (a.heads + 15) / 16, splits), 128, smem, ctx().stream>>>(t, a, QA, ldqa, cache, part, R);
-    GTB_LAUNCHED();
-    return GTB_OK;
-}
-// -1: sizes outside the kernel (the caller takes the row kernels)
-int lat_dec_mma(const PassTables& t, const SoftAttn& a, int R, int splits, const float* QA, int ldqa, const bf16* cache, float* part) {
-    if (a.vdim <= 128) return launch_lat_dec_mma<32>(t, a, R, splits, QA, ldqa, cache, part);
-    if (a.vdim <= 256) return launch_lat_dec_mma<64>(t, a, R, splits, QA, ldqa, cache, part);
-    if (a.vdim <= 512) return launch_lat_dec_mma<128>(t, a, R, splits, QA, ldqa, cache, part);
-    return -1;
-}
-
 // One pre-norm layer on R rows.  pend carries the update of the sublayer before it (none for the first layer) and leaves with this
 // layer's last sublayer pending; cap_prev: where the sum of the copies after the previous layer goes (capture), or null.
 template <typename OT>
@@ -745,86 +945,8 @@ int run_prenorm_layer(gtb_seq_model* m, const PassTables& t, int R, int S, const
     if (rc) return rc;
     rc = product<OT>(m, opA, wp, l.w_mix, wp, m->P, l.n1, R, l.n1, wp, nullptr, 0);
     if (rc) return rc;
-    const BranchW& b = l.br[0];
-    // prompt portions in bf16 mode: keys and values of the visible range are expanded from the cached latents and the heads run the
-    // tensor-core softmax attention; everything else runs the absorbed form on the row kernels
-    const bool expand = portions && sizeof(OT) == 2 && seg_slots && m->latKx && b.d.dim + b.d.rope_dim <= 128 && b.d.vdim <= 128;
-    {
-        const LatAttn a = lat_args(m, b);
-        const int hd = a.dim + a.rope;
-        k_lat_prep<OT><<<dim3(R, a.q_rank > 0 ? 2 : 1), 128, 0, st>>>(t, a, m->P, l.n1, (OT*)run.kc[0], (OT*)m->opQ, b.qrank_p);
-        GTB_LAUNCHED();
-        const float* Q = m->P;
-        int ldq = l.n1, q0 = b.q_off;
-        if (a.q_rank > 0) {
-            ldq = a.heads * hd + a.heads;         // room for the heads' gate logits behind the queries (the tiled path reads them there)
-            rc = product<OT>(m, m->opQ, b.qrank_p, b.w_uq, b.qrank_p, m->latQ, ldq, R, a.heads * hd, b.qrank_p, nullptr, 0);
-            if (rc) return rc;
-            Q = m->latQ; q0 = 0;
-        }
-        if (expand) {
-            const int ld_qr = a.heads * hd + a.heads, nx = a.heads * (a.dim + a.vdim);
-            k_lat_qrot<<<R, 128, 0, st>>>(t, a, Q, ldq, q0, m->P, l.n1, m->latQ, ld_qr);
-            GTB_LAUNCHED();
-            for (int s = 0; s < S; s++) {
-                const int slot = seg_slots[s], p0 = m->host_pos[slot];
-                const int lo = b.d.window > 0 ? std::max(0, p0 - b.d.window + 1) : 0, n = p0 + seg_lens[s] - lo;
-                const bf16* src = (const bf16*)run.kc[0] + ((size_t)slot * c.max_ctx + lo) * b.c_ld;
-                rc = product<OT>(m, src, b.c_ld, b.w_uk, b.rank_p, m->latX, nx, n, nx, b.rank_p, nullptr, 0);      // uk and uv rows are one matrix
-                if (rc) return rc;
-                k_lat_pack<<<n, 256, 0, st>>>(a, m->latX, n, slot, lo, (const bf16*)run.kc[0], m->latKx, m->latVx);
-                GTB_LAUNCHED();
-            }
-            SoftAttn sa{};
-            sa.heads = sa.kv_heads = a.heads; sa.dim = hd; sa.vdim = a.vdim; sa.scale = b.d.scale; sa.eps = c.eps; sa.window = b.d.window; sa.sink = b.d_sink;
-            sa.gate = b.d.gated; sa.q_off = 0; sa.g_off = a.heads * hd; sa.a_off = b.a_off; sa.own_kv = 1; sa.max_ctx = c.max_ctx;
-            rc = sattn_mma(t, sa, S, n_qtiles, m->latQ, ld_qr, m->latKx, m->latVx, nullptr, nullptr, (bf16*)opC, l.kout_p);
-            if (rc > 0) return rc;
-            if (rc < 0) return gtb::fail(GTB_ERR_STATE, "head sizes outside the tiled attention kernel");
-        }
-    }
-    if (!expand) {
-        const LatAttn a = lat_args(m, b);
-        const int hd = a.dim + a.rope;
-        const float* Q = a.q_rank > 0 ? m->latQ : m->P;
-        const int ldq = a.q_rank > 0 ? a.heads * hd + a.heads : l.n1, q0 = a.q_rank > 0 ? 0 : b.q_off;
-        k_lat_qabs<<<dim3(R, a.heads, (a.rank + 127) / 128), 128, (hd + 512) * sizeof(float), st>>>(t, a, Q, ldq, q0, b.w_uk, b.rank_p, m->latQA);
-        GTB_LAUNCHED();
-        const SoftAttn sa = lat_soft_args(m, b);
-        const int ldqa = a.heads * sa.dim, ld_ol = (a.heads * a.rank + 7) / 8 * 8;
-        const size_t smem = (sa.dim + 128 + 33) * sizeof(float);
-        bool done = false;
-        if (sizeof(OT) == 2 && m->fused_attn && !portions && R <= SPLIT_MAX_ROWS && m->sattn_part) {
-            // decode rows in bf16 mode: 16 heads per CTA on tensor cores, one CTA per 64 keys of the longest key list this layer can meet
-            const int max_keys = sa.window > 0 ? std::min(c.max_ctx, sa.window) : c.max_ctx;
-            const int splits = std::max(1, std::min(32, (max_keys + 63) / 64));
-            rc = lat_dec_mma(t, sa, R, splits, m->latQA, ldqa, (const bf16*)run.kc[0], m->sattn_part);
-            if (rc > 0) return rc;
-            if (rc == 0) {
-                k_sattn_join<OT><<<dim3(R, sa.heads), 128, 0, st>>>(sa, m->latQA, ldqa, m->sattn_part, R, splits, (OT*)m->opO, ld_ol);
-                GTB_LAUNCHED();
-                done = true;
-            }
-        }
-        if (!done && !portions && R <= SPLIT_MAX_ROWS && m->sattn_part) {
-            const int max_keys = sa.window > 0 ? std::min(c.max_ctx, sa.window) : c.max_ctx;
-            const int splits = std::max(1, std::min(32, (max_keys + 127) / 128));
-            if (splits > 1) {
-                k_sattn_split<OT><<<dim3(R, sa.heads, splits), 128, smem, st>>>(t, sa, m->latQA, ldqa, (const OT*)run.kc[0], (const OT*)run.kc[0], nullptr, nullptr, m->sattn_part, R);
-                GTB_LAUNCHED();
-                k_sattn_join<OT><<<dim3(R, sa.heads), 128, 0, st>>>(sa, m->latQA, ldqa, m->sattn_part, R, splits, (OT*)m->opO, ld_ol);
-                GTB_LAUNCHED();
-                done = true;
-            }
-        }
-        if (!done) {
-            k_sattn<OT><<<dim3(R, sa.heads), 128, smem, st>>>(t, sa, m->latQA, ldqa, (const OT*)run.kc[0], (const OT*)run.kc[0], nullptr, nullptr, (OT*)m->opO, ld_ol);
-            GTB_LAUNCHED();
-        }
-        const int n_out = a.heads * a.vdim;
-        k_lat_vup<OT><<<dim3(R, std::max(1, std::min(std::max(1, 4096 / R), (n_out + 7) / 8))), 256, 0, st>>>(a, (const OT*)m->opO, ld_ol, b.w_uv, b.rank_p, m->P, l.n1, b.d.gated, opC, l.kout_p);
-        GTB_LAUNCHED();
-    }
+    rc = run_latent_branch<OT>(m, t, R, S, run, l, portions, seg_lens, seg_slots, n_qtiles);
+    if (rc) return rc;
     rc = product<OT>(m, opC, l.kout_p, l.w_out, l.kout_p, m->Y, W, R, W, l.kout_p, nullptr, 0);
     if (rc) return rc;
     pend.Y = m->Y; pend.hc = l.hc[0];
@@ -924,7 +1046,7 @@ int run_pass(gtb_seq_model* m, const PassTables& t, int R, int S, bool from_pend
                                        m->prenorm ? m->xs : m->x, c.loop_times > 0 ? m->x0 : nullptr, first_reads_x ? opA : (OT*)nullptr, wp);
         GTB_LAUNCHED();
         if (m->sandwich) {
-            k_norm_rows<OT><<<R, 256, 0, st>>>(m->x, W, sw_norm(m, m->L[m->runs[0].layer], 0), nullptr, opA, wp);
+            k_norm_rows<OT><<<R, 256, 0, st>>>(m->x, W, sw_norm(m, m->L[m->runs[0].layer], 0), nullptr, opA, wp, 1.0f);
             GTB_LAUNCHED();
         }
     }
@@ -935,7 +1057,7 @@ int run_pass(gtb_seq_model* m, const PassTables& t, int R, int S, bool from_pend
         const LayerW& l = m->L[run.layer];
         if (l.d.style == GTB_BLOCK_SANDWICH) {
             const NormArgs next = u + 1 < m->runs.size() ? sw_norm(m, m->L[m->runs[u + 1].layer], 0) : NormArgs{};
-            int rc = run_sandwich_layer<OT>(m, t, R, S, run, l, portions, seg_lens, n_qtiles, next);
+            int rc = run_sandwich_layer<OT>(m, t, R, S, run, l, portions, seg_lens, seg_slots, n_qtiles, next);
             if (rc) return rc;
             if (m->capture) {
                 GTB_CUDA(cudaMemcpyAsync(m->cap + u * (size_t)m->max_rows * W, m->x, (size_t)R * W * sizeof(float), cudaMemcpyDeviceToDevice, st));
@@ -989,7 +1111,7 @@ int run_pass(gtb_seq_model* m, const PassTables& t, int R, int S, bool from_pend
                 GTB_LAUNCHED();
             }
             if (c.taps > 1) {
-                k_canon_tail<<<dim3(S, (W + 255) / 256), 256, 0, st>>>(t, m->h, W, c.taps, run.tail);
+                k_canon_tail<<<dim3(S, (W + 255) / 256), 256, 0, st>>>(t, m->h, W, W, c.taps, run.tail);
                 GTB_LAUNCHED();
             }
         } else {
@@ -1052,10 +1174,12 @@ int run_pass(gtb_seq_model* m, const PassTables& t, int R, int S, bool from_pend
         }
     }
     if (n_want > 0) {
-        if (c.final_norm == 3) {
+        float ls = c.logit_scale != 0.0f ? c.logit_scale : 1.0f;        // what is left of the logit scale for the logits themselves
+        if (c.final_norm >= 3) {
             NormArgs fn{};
             fn.kind = GTB_NORM_LAYER; fn.w = m->final_gain; fn.b = m->final_b; fn.eps = c.eps;
-            k_norm_rows<OT><<<n_want, 256, 0, st>>>(m->x, W, fn, d_want, opH, wp);
+            k_norm_rows<OT><<<n_want, 256, 0, st>>>(m->x, W, fn, d_want, opH, wp, ls);      // the product is linear: the scale rides on its operand
+            ls = 1.0f;
         } else if (c.final_norm == 2) {
             NormArgs fn{};
             fn.kind = GTB_NORM_DYT; fn.w = m->final_gain; fn.b = m->final_b; fn.alpha = m->final_a;
@@ -1065,9 +1189,9 @@ int run_pass(gtb_seq_model* m, const PassTables& t, int R, int S, bool from_pend
         GTB_LAUNCHED();
         int rc = product<OT>(m, opH, wp, m->head, wp, m->logits, c.vocab, n_want, c.vocab, wp, nullptr, 0);
         if (rc) return rc;
-        if (c.logit_softcap > 0.0f) {
+        if (c.logit_softcap > 0.0f || ls != 1.0f) {
             const size_t n = (size_t)n_want * c.vocab;
-            k_softcap<<<(unsigned)((n + 255) / 256), 256, 0, st>>>(m->logits, n, c.logit_softcap);
+            k_logits_post<<<(unsigned)((n + 255) / 256), 256, 0, st>>>(m->logits, n, ls, c.logit_softcap);
             GTB_LAUNCHED();
         }
     }
@@ -1112,9 +1236,13 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
         TRY(dalloc_t(m, &m->bigram, (size_t)(c.bigram_buckets + 1) * W));
         want_matrix(m, "bigram", m->bigram, c.bigram_buckets + 1, W, W);
     }
-    TRY(dalloc_t(m, &m->head, (size_t)c.vocab * wp));
-    want_matrix(m, "head", m->head, c.vocab, W, wp);
-    REQ(c.final_norm >= 0 && c.final_norm <= 3);
+    if (c.tied_head && wp == W) m->head = m->embed;
+    else {
+        TRY(dalloc_t(m, &m->head, (size_t)c.vocab * wp));
+        if (c.tied_head) { TensorDest& d = m->tensors["embed"]; d.also = m->head; d.also_ld = wp; }     // the product wants padded rows: a copy of its own
+        else want_matrix(m, "head", m->head, c.vocab, W, wp);
+    }
+    REQ(c.final_norm >= 0 && c.final_norm <= 4);
     REQ(c.streams >= 0 && c.streams <= HC_MAX && c.logit_softcap >= 0.0f);
     TRY(dalloc_t(m, &m->final_gain, c.final_norm ? W : 1));
     if (c.final_norm) want_vector(m, "final.norm", m->final_gain, W, 0);
@@ -1154,8 +1282,10 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
         REQ(sw == m->sandwich);                  // a sandwich layer hands its successor a normalised operand
         REQ(!(pre || sw) || (c.loop_times == 0 && c.taps == 0));
         REQ(l.d.n_branches >= 1 && l.d.n_branches <= (post || pre ? 1 : 2));
+        if (l.d.n_branches == 2) for (const gtb_seq_branch& d : l.d.branch) REQ(d.kind != GTB_MIX_LATENT_ATTN && d.out_bias == 0);
         REQ(l.d.ff >= 0);
-        if (sw) REQ((l.d.norm_kind == GTB_NORM_RMS || l.d.norm_kind == GTB_NORM_LAYER) && (l.d.ff == 0 || l.d.ff_kind == GTB_FF_SWIGLU || l.d.ff_kind == GTB_FF_GROUP_EXPERTS));
+        if (sw) REQ((l.d.norm_kind == GTB_NORM_RMS || l.d.norm_kind == GTB_NORM_LAYER || l.d.norm_kind == GTB_NORM_LAYER_NB) &&
+                    (l.d.ff == 0 || l.d.ff_kind == GTB_FF_SWIGLU || l.d.ff_kind == GTB_FF_GROUP_EXPERTS || l.d.ff_kind == GTB_FF_GELU));
         else if (pre) REQ((l.d.norm_kind == GTB_NORM_RMS || l.d.norm_kind == GTB_NORM_DYT) && (l.d.ff == 0 || l.d.ff_kind == GTB_FF_GEGLU || l.d.ff_kind == GTB_FF_GATED_EXPERTS));
         else REQ(post ? (l.d.ff == 0 || l.d.ff_kind == GTB_FF_POLYNORM || l.d.ff_kind == GTB_FF_EXPERTS) : l.d.ff_kind == GTB_FF_GEGLU);
         l.ff = l.d.ff;
@@ -1166,25 +1296,33 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
             b.d = l.d.branch[bi];
             gtb_seq_branch& d = b.d;
             REQ(pre ? d.kind == GTB_MIX_LATENT_ATTN : post ? (d.kind == GTB_MIX_MINGRU || d.kind == GTB_MIX_SOFTMAX_ATTN) :
-                sw ? (d.kind == GTB_MIX_SOFTMAX_ATTN || d.kind == GTB_MIX_RETENTION) : (d.kind == GTB_MIX_SIGMOID_ATTN || d.kind == GTB_MIX_RETENTION));
+                sw ? (d.kind == GTB_MIX_SOFTMAX_ATTN || d.kind == GTB_MIX_RETENTION || d.kind == GTB_MIX_LATENT_ATTN) : (d.kind == GTB_MIX_SIGMOID_ATTN || d.kind == GTB_MIX_RETENTION));
+            REQ(d.rot_scaling == GTB_ROT_SCALE_WAVES || d.rot_scaling == GTB_ROT_SCALE_YARN);
+            if (d.rot_factor > 0.0f) REQ(d.rot_original > 0.0f && d.rot_base > 1.0f && d.rot_low > 0.0f && d.rot_high > 0.0f);
+            if (!sw || d.kind != GTB_MIX_SOFTMAX_ATTN) REQ(d.conv == 0 && d.v_from_k == 0 && d.keep_first == 0 && d.slopes == 0);
+            REQ(d.out_bias == 0 || (sw && d.kind != GTB_MIX_RETENTION));
             if (d.kind == GTB_MIX_LATENT_ATTN) {
                 REQ(d.heads > 0 && d.dim > 0 && d.rope_dim >= 0 && d.vdim > 0 && d.kv_rank > 0 && d.q_rank >= 0 && d.window >= 0);
                 REQ(d.kv_rank <= 512 && d.kv_rank + d.rope_dim <= 1024);        // the absorbed form runs on the row kernels of softmax attention
-                REQ(d.rot_dims >= 0 && d.rot_dims <= d.rope_dim && d.rot_dims % 2 == 0 && (d.gated == 0 || d.gated == 3));
-                d.kv_heads = 1; d.kv_from = -1; d.pool = 0;
+                REQ(d.rot_dims >= 0 && d.rot_dims <= d.rope_dim && d.rot_dims % 2 == 0 && (d.gated == 0 || d.gated == 2 || d.gated == 3) && d.sink <= 1);
+                REQ(d.kv_from < i);
+                if (d.kv_from >= 0) {
+                    REQ(c.loop_times == 0);
+                    const LayerW& src = m->L[d.kv_from];
+                    const gtb_seq_branch& sd = src.br[0].d;
+                    REQ(src.d.style == l.d.style && src.d.n_branches == 1 && sd.kind == GTB_MIX_LATENT_ATTN && sd.kv_from < 0);
+                    REQ(sd.kv_rank == d.kv_rank && sd.rope_dim == d.rope_dim && sd.rot_dims == d.rot_dims && sd.rot_layout == d.rot_layout && sd.rot_base == d.rot_base);
+                    REQ(sd.rot_factor == d.rot_factor && sd.rot_scaling == d.rot_scaling && sd.rot_low == d.rot_low && sd.rot_high == d.rot_high && sd.rot_original == d.rot_original);
+                } else d.kv_from = -1;
+                d.kv_heads = 1; d.pool = 0;
                 const int hd = d.dim + d.rope_dim, nq = d.q_rank > 0 ? d.q_rank : d.heads * hd;
-                b.q_off = n1; b.kv_off = n1 + nq; b.g_off = b.kv_off + d.kv_rank + d.rope_dim;
-                n1 = b.g_off + (d.gated ? d.heads : 0);
+                b.q_off = n1; b.kv_off = n1 + nq; b.g_off = b.kv_off + (d.kv_from < 0 ? d.kv_rank + d.rope_dim : 0);
+                n1 = b.g_off + (d.gated == 2 ? d.heads * d.vdim : d.gated ? d.heads : 0);
                 b.a_off = ko; ko += d.heads * d.vdim;
                 b.rank_p = pad64(d.kv_rank); b.qrank_p = d.q_rank > 0 ? pad64(d.q_rank) : 0;
                 b.c_ld = std::max((d.kv_rank + d.rope_dim + 7) / 8 * 8, b.rank_p);
-                if (d.rot_dims > 0) {
-                    b.inv_freq.resize(d.rot_dims / 2);
-                    for (int k = 0; k < d.rot_dims / 2; k++) b.inv_freq[k] = (float)pow((double)d.rot_base, -2.0 * k / d.rot_dims);
-                    TRY(dalloc_t(m, &b.d_inv_freq, b.inv_freq.size()));
-                    GTB_CUDA(cudaMemcpyAsync(b.d_inv_freq, b.inv_freq.data(), b.inv_freq.size() * sizeof(float), cudaMemcpyHostToDevice, ctx().stream));
-                }
-                m->lat_q_max = std::max(m->lat_q_max, d.heads * hd + d.heads);
+                TRY(upload_rot_table(m, b));
+                m->lat_q_max = std::max(m->lat_q_max, d.heads * hd);
                 if (hd <= 128 && d.vdim <= 128) {
                     m->lat_kx_max = std::max(m->lat_kx_max, d.heads * hd);
                     m->lat_vx_max = std::max(m->lat_vx_max, d.heads * d.vdim);
@@ -1213,37 +1351,33 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
             if (d.kind == GTB_MIX_SOFTMAX_ATTN) {
                 REQ(d.qk_norm >= 0 && d.qk_norm <= 3 && d.gated >= 0 && d.gated <= 3 && d.window >= 0 && d.pool >= 0 && d.softcap >= 0.0f);
                 REQ(d.maps <= 2 && d.chunk >= 0 && d.rot_divide >= 0.0f && (d.gated != 3 || sw));
-                if (d.maps == 2) REQ(d.pool == 0 && d.sink == 0 && (d.gated == 0 || d.gated == 3));
+                if (d.maps == 2) REQ(d.pool == 0 && d.sink == 0 && (d.gated == 0 || d.gated == 3) && d.v_from_k == 0 && d.conv == 0);
+                REQ(d.sink >= 0 && d.sink <= (sw ? 2 : 1));
+                REQ(d.conv >= 0 && d.conv <= 64 && (d.conv == 0 || (d.qk_norm == 0 && d.rot_dims == 0)));
+                REQ(!d.v_from_k || d.dim == d.vdim);
+                REQ(d.keep_first >= 0 && ((d.keep_first == 0 && d.slopes == 0) || d.pool == 0));
                 if (!sw) d.out_scale = 1.0f;
                 REQ(d.kv_from < i);
                 if (d.kv_from >= 0) {
                     REQ(c.loop_times == 0);
                     const LayerW& src = m->L[d.kv_from];
                     REQ(src.d.style == l.d.style && src.d.n_branches == 1 && src.br[0].d.kind == GTB_MIX_SOFTMAX_ATTN && src.br[0].d.kv_from < 0);
-                    REQ(src.br[0].d.kv_heads == d.kv_heads && src.br[0].d.dim == d.dim && src.br[0].d.vdim == d.vdim && src.br[0].d.maps == d.maps);
+                    REQ(src.br[0].d.kv_heads == d.kv_heads && src.br[0].d.dim == d.dim && src.br[0].d.vdim == d.vdim && src.br[0].d.maps == d.maps && src.br[0].d.v_from_k == d.v_from_k);
                     REQ(l.d.n_branches == 1);
                 } else d.kv_from = -1;
                 b.q_off = n1; n1 += b.kq;
-                if (d.kv_from < 0) { b.k_off = n1; n1 += b.kk; b.v_off = n1; n1 += b.kv; }
+                if (d.kv_from < 0) { b.k_off = n1; n1 += b.kk; b.v_off = n1; if (!d.v_from_k) n1 += b.kv; }
                 if (d.gated) { b.g_off = n1; n1 += d.gated == 3 ? d.heads : d.heads * d.vdim; }
                 b.a_off = ko; ko += d.heads * d.vdim;
                 if (d.maps == 2) m->ro_max = std::max(m->ro_max, 2 * d.heads * d.vdim);
-                if (d.rot_dims > 0) {
-                    // frequencies in double, rounded once: base^(-2k/dims); long wavelengths slowed down by rot_factor, a linear blend between
-                    b.inv_freq.resize(d.rot_dims / 2);
-                    for (int k = 0; k < d.rot_dims / 2; k++) {
-                        double f = pow((double)d.rot_base, -2.0 * k / d.rot_dims);
-                        if (d.rot_factor > 0.0f) {
-                            const double wl = 2.0 * M_PI / f, orig = d.rot_original, lo = d.rot_low, hi = d.rot_high, fac = d.rot_factor;
-                            if (wl > orig / lo) f = f / fac;
-                            else if (!(wl < orig / hi)) { const double sm = (orig / wl - lo) / (hi - lo); f = (1.0 - sm) * f / fac + sm * f; }
-                        }
-                        if (d.rot_divide > 0.0f) f /= (double)d.rot_divide;
-                        b.inv_freq[k] = (float)f;
-                    }
-                    TRY(dalloc_t(m, &b.d_inv_freq, b.inv_freq.size()));
-                    GTB_CUDA(cudaMemcpyAsync(b.d_inv_freq, b.inv_freq.data(), b.inv_freq.size() * sizeof(float), cudaMemcpyHostToDevice, ctx().stream));
+                TRY(upload_rot_table(m, b));
+                if (d.slopes) {
+                    b.slopes.resize(d.heads);
+                    for (int h = 0; h < d.heads; h++) b.slopes[h] = (float)exp2(-8.0 * (h + 1) / d.heads);
+                    TRY(dalloc_t(m, &b.d_slope, d.heads));
+                    GTB_CUDA(cudaMemcpyAsync(b.d_slope, b.slopes.data(), d.heads * sizeof(float), cudaMemcpyHostToDevice, ctx().stream));
                 }
+                if (d.conv > 0) m->conv_q_max = std::max(m->conv_q_max, b.kq);
                 continue;
             }
             b.q_off = n1; b.k_off = n1 + b.kq; b.v_off = b.k_off + b.kk; n1 = b.v_off + b.kv;
@@ -1257,13 +1391,8 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
                 d.decay = nullptr;
                 TRY(dalloc_t(m, &b.d_decay, d.heads));
                 GTB_CUDA(cudaMemcpyAsync(b.d_decay, b.decay.data(), d.heads * sizeof(float), cudaMemcpyHostToDevice, ctx().stream));
-                if (d.rot_dims > 0) {
-                    // (same stream as the allocation's zero fill: a copy on another stream could be overtaken by it)
-                    b.inv_freq.resize(d.rot_dims / 2);
-                    for (int k = 0; k < d.rot_dims / 2; k++) b.inv_freq[k] = (float)pow((double)d.rot_base, -2.0 * k / d.rot_dims);
-                    TRY(dalloc_t(m, &b.d_inv_freq, b.inv_freq.size()));
-                    GTB_CUDA(cudaMemcpyAsync(b.d_inv_freq, b.inv_freq.data(), b.inv_freq.size() * sizeof(float), cudaMemcpyHostToDevice, ctx().stream));
-                }
+                REQ(d.rot_factor == 0.0f);
+                TRY(upload_rot_table(m, b));
             }
         }
         GTB_CUDA(cudaStreamSynchronize(ctx().stream));       // the vectors above are read from members that may move; wait for the copies
@@ -1297,28 +1426,31 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
                 } else {
                     want_matrix(m, bp + "q", l.w_mix + (size_t)b.q_off * wp, d.heads * hd, W, wp);
                 }
-                want_matrix(m, bp + "dkv", l.w_mix + (size_t)b.kv_off * wp, d.kv_rank + d.rope_dim, W, wp);
-                TRY(dalloc_t(m, &b.d_kvnorm, d.kv_rank));
-                want_vector(m, bp + "dkv.norm", b.d_kvnorm, d.kv_rank, 0);
+                if (d.kv_from < 0) {
+                    want_matrix(m, bp + "dkv", l.w_mix + (size_t)b.kv_off * wp, d.kv_rank + d.rope_dim, W, wp);
+                    TRY(dalloc_t(m, &b.d_kvnorm, d.kv_rank));
+                    want_vector(m, bp + "dkv.norm", b.d_kvnorm, d.kv_rank, 0);
+                }
                 TRY(dalloc_t(m, &b.w_uk, (size_t)d.heads * (d.dim + d.vdim) * b.rank_p));      // uv follows uk: one product expands keys and values
                 b.w_uv = b.w_uk + (size_t)d.heads * d.dim * b.rank_p;
                 want_matrix(m, bp + "uk", b.w_uk, d.heads * d.dim, d.kv_rank, b.rank_p);
                 want_matrix(m, bp + "uv", b.w_uv, d.heads * d.vdim, d.kv_rank, b.rank_p);
                 if (d.sink) { TRY(dalloc_t(m, &b.d_sink, d.heads)); want_vector(m, bp + "sink", b.d_sink, d.heads, 0); }
-                if (d.gated) want_matrix(m, bp + "g", l.w_mix + (size_t)b.g_off * wp, d.heads, W, wp);
+                if (d.gated) want_matrix(m, bp + "g", l.w_mix + (size_t)b.g_off * wp, d.gated == 2 ? d.heads * d.vdim : d.heads, W, wp);
                 want_matrix(m, bp + "o", l.w_out + b.a_off, W, d.heads * d.vdim, l.kout_p);
+                if (d.out_bias) { TRY(dalloc_t(m, &l.d_obias, W)); want_vector(m, bp + "o.b", l.d_obias, W, 0); }
                 continue;
             }
             want_matrix(m, bp + "q", l.w_mix + (size_t)b.q_off * wp, b.kq, W, wp);
             const bool own_kv = !(d.kind == GTB_MIX_SOFTMAX_ATTN && d.kv_from >= 0);
             if (own_kv) {
                 want_matrix(m, bp + "k", l.w_mix + (size_t)b.k_off * wp, b.kk, W, wp);
-                want_matrix(m, bp + "v", l.w_mix + (size_t)b.v_off * wp, b.kv, W, wp);
+                if (!d.v_from_k) want_matrix(m, bp + "v", l.w_mix + (size_t)b.v_off * wp, b.kv, W, wp);
             }
             if (d.bias) {                           // bias vectors of the fused projection; columns without one stay zero
                 if (!l.d_bias) TRY(dalloc_t(m, &l.d_bias, n1));
                 want_vector(m, bp + "q.b", l.d_bias + b.q_off, b.kq, 0);
-                if (own_kv) { want_vector(m, bp + "k.b", l.d_bias + b.k_off, b.kk, 0); want_vector(m, bp + "v.b", l.d_bias + b.v_off, b.kv, 0); }
+                if (own_kv) { want_vector(m, bp + "k.b", l.d_bias + b.k_off, b.kk, 0); if (!d.v_from_k) want_vector(m, bp + "v.b", l.d_bias + b.v_off, b.kv, 0); }
             }
             if ((d.kind == GTB_MIX_RETENTION || d.kind == GTB_MIX_SOFTMAX_ATTN) && d.gated)
                 want_matrix(m, bp + "g", l.w_mix + (size_t)b.g_off * wp, (d.kind == GTB_MIX_SOFTMAX_ATTN && d.gated == 3) ? d.heads : d.heads * d.vdim, W, wp);
@@ -1344,7 +1476,17 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
                     const char* nm[4] = {"lq1", "lk1", "lq2", "lk2"};
                     for (int q = 0; q < 4; q++) { TRY(dalloc_t(m, &b.d_lam[q], d.dim)); want_vector(m, bp + nm[q], b.d_lam[q], d.dim, 0); }
                 }
-                if (d.sink) { TRY(dalloc_t(m, &b.d_sink, d.heads)); want_vector(m, bp + "sink", b.d_sink, d.heads, 0); }
+                if (d.sink) {                       // sink 2: score 0 for every head, the allocation's zero fill
+                    TRY(dalloc_t(m, &b.d_sink, d.heads));
+                    if (d.sink == 1) want_vector(m, bp + "sink", b.d_sink, d.heads, 0);
+                }
+                if (d.conv > 0) {                   // one table: query channels, then key channels
+                    const int nk = own_kv ? b.kk : 0;
+                    TRY(dalloc_t(m, &b.d_conv, (size_t)(b.kq + nk) * d.conv));
+                    want_vector(m, bp + "q.conv", b.d_conv, b.kq, d.conv);
+                    if (own_kv) want_vector(m, bp + "k.conv", b.d_conv + (size_t)b.kq * d.conv, nk, d.conv);
+                }
+                if (d.out_bias) { TRY(dalloc_t(m, &l.d_obias, W)); want_vector(m, bp + "o.b", l.d_obias, W, 0); }
             }
         }
         if (sw) {
@@ -1367,6 +1509,13 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
                         for (const char* nm : {"mlp.gate", "mlp.up"}) { TensorDest& d = m->tensors[lp + nm]; d.group = 32; d.group_stride = 64; }
                     want_matrix(m, lp + "mlp.down", l.w_down, W, l.ff, l.kfp);
                     m->g_cols = std::max(m->g_cols, 2 * l.ff);
+                    m->kout_p_max = std::max(m->kout_p_max, l.kfp);
+                } else if (l.d.ff_kind == GTB_FF_GELU) {
+                    TRY(dalloc_t(m, &l.w_up, (size_t)l.ff * wp));
+                    TRY(dalloc_t(m, &l.w_down, (size_t)W * l.kfp));
+                    want_matrix(m, lp + "mlp.up", l.w_up, l.ff, W, wp);
+                    want_matrix(m, lp + "mlp.down", l.w_down, W, l.ff, l.kfp);
+                    m->g_cols = std::max(m->g_cols, l.ff);
                     m->kout_p_max = std::max(m->kout_p_max, l.kfp);
                 } else {
                     const int E = l.d.experts, G = std::max(1, l.d.route_groups), keep = l.d.route_keep > 0 ? l.d.route_keep : G;
@@ -1552,6 +1701,7 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
         for (int bi = 0; bi < l.d.n_branches; bi++) {
             const gtb_seq_branch& d = l.br[bi].d;
             if (d.kind == GTB_MIX_LATENT_ATTN) {
+                if (d.kv_from >= 0) { r.kc[bi] = m->runs[d.kv_from].kc[0]; continue; }      // no loop (checked above): run j is layer j
                 const size_t cb = (size_t)c.max_ctx * l.br[bi].c_ld * es;
                 TRY(dalloc(m, &r.kc[bi], cb * c.n_slots));
                 per_slot += cb;
@@ -1563,8 +1713,15 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
                 } else {
                     const size_t kb = (size_t)c.max_ctx * d.kv_heads * std::max(1, d.maps) * d.dim * es, vb = (size_t)c.max_ctx * d.kv_heads * d.vdim * es;
                     TRY(dalloc(m, &r.kc[bi], kb * c.n_slots));
-                    TRY(dalloc(m, &r.vc[bi], vb * c.n_slots));
-                    per_slot += kb + vb;
+                    if (d.v_from_k) r.vc[bi] = r.kc[bi];
+                    else TRY(dalloc(m, &r.vc[bi], vb * c.n_slots));
+                    per_slot += d.v_from_k ? kb : kb + vb;
+                }
+                if (d.conv > 1) {
+                    REQ(!r.ctail);                              // one convolved branch per layer
+                    r.ctail_n = (d.conv - 1) * (l.br[bi].kq + (d.kv_from < 0 ? l.br[bi].kk : 0));
+                    TRY(dalloc_t(m, &r.ctail, (size_t)c.n_slots * r.ctail_n));
+                    per_slot += r.ctail_n * sizeof(float);
                 }
                 if (d.kind == GTB_MIX_SOFTMAX_ATTN && d.window > 0 && d.pool > 0) {      // pooled blocks follow this layer's own block size
                     r.max_blocks = c.max_ctx / d.pool + 1;
@@ -1635,10 +1792,13 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
         m->attn_splits = std::max(1, std::min(32, c.max_ctx / 128));
         if (hv > 0 && m->attn_splits > 1) TRY(dalloc_t(m, &m->attn_part, (size_t)m->attn_splits * SPLIT_MAX_ROWS * hv));
     }
+    if (m->conv_q_max > 0) TRY(dalloc_t(m, &m->convQ, R * m->conv_q_max));
     if (m->prenorm) {
         TRY(dalloc_t(m, &m->xs, (size_t)m->ns * R * W));
         TRY(dalloc_t(m, &m->Y2, R * W));
         TRY(dalloc_t(m, &m->shw, R));
+    }
+    if (m->lat_q_max > 0) {
         TRY(dalloc_t(m, &m->latQ, R * std::max(m->lat_q_max, 1)));
         TRY(dalloc_t(m, &m->latQA, R * std::max(m->lat_qa_max, 1)));
         TRY(dalloc(m, &m->opQ, R * std::max(m->lat_qr_max, 8) * es));
@@ -1706,6 +1866,7 @@ int gtb_seq_set_tensor(gtb_seq_t m, const char* name, const void* h_bf16, const 
                                       (size_t)std::min(d.split_cols, d.cols - c0) * 2, d.rows, cudaMemcpyHostToDevice));
         } else {
             GTB_CUDA(cudaMemcpy2D(d.dst, (size_t)d.ld * 2, h_bf16, (size_t)d.cols * 2, (size_t)d.cols * 2, d.rows, cudaMemcpyHostToDevice));
+            if (d.also) GTB_CUDA(cudaMemcpy2D(d.also, (size_t)d.also_ld * 2, h_bf16, (size_t)d.cols * 2, (size_t)d.cols * 2, d.rows, cudaMemcpyHostToDevice));
         }
     } else {
         const size_t n = d.scalar ? 1 : (size_t)d.rows * std::max(d.cols, 1);
@@ -1742,6 +1903,7 @@ int gtb_seq_slot_reset(gtb_seq_t m, int slot) {
                 const size_t sb = state_floats(l.br[bi].d) * sizeof(float);
                 GTB_CUDA(cudaMemsetAsync((char*)r.state[bi] + sb * slot, 0, sb, st));
             }
+        if (r.ctail) GTB_CUDA(cudaMemsetAsync(r.ctail + (size_t)r.ctail_n * slot, 0, r.ctail_n * sizeof(float), st));
         if (r.tail) {
             const size_t tb = (size_t)(m->cfg.taps - 1) * m->cfg.width * sizeof(float);
             GTB_CUDA(cudaMemsetAsync((char*)r.tail + tb * slot, 0, tb, st));

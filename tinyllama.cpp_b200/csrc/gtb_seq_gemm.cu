@@ -18,7 +18,8 @@
 //
 // Grouped products (routed experts): the rows of A are sorted into groups that start on multiples of 128 rows, a device table gives
 // every M tile its group (or -1: nothing to do), and group g multiplies with rows [g N, (g + 1) N) of W.  EPI_RELU2 writes
-// row_w[row] * relu(acc)^2 as a bf16 operand block (the expert's activation, already weighted with the router's score).
+// row_w[row] * relu(acc)^2 as a bf16 operand block (the expert's activation, already weighted with the router's score); EPI_GELU writes
+// gelu(acc) (erf form), the activation of an ungated feed-forward, the same way.
 #include "gtb_seq_gemm.h"
 
 #include <cuda_bf16.h>
@@ -30,7 +31,7 @@ namespace gtb {
 namespace seq {
 
 constexpr int SQ_BM = 128, SQ_BK = 64, SQ_THREADS = 320, SQ_EPI_THREADS = 256;
-enum { SQ_EPI_F32 = 0, SQ_EPI_GEGLU = 1, SQ_EPI_RELU2 = 2 };
+enum { SQ_EPI_F32 = 0, SQ_EPI_GEGLU = 1, SQ_EPI_RELU2 = 2, SQ_EPI_GELU = 3 };
 
 template <int BN> struct SqCfg {
     static constexpr int STAGES = (BN == 256) ? 4 : 6;
@@ -77,6 +78,19 @@ __device__ __forceinline__ float sq_gelu(float z) {
 
 // silu(z) = z / (1 + 2^(-z log2 e)) on the special-function unit; the value is rounded to bf16 right after
 __device__ __forceinline__ float sq_silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+// gelu(z) = z (1 + erf(z / sqrt 2)) / 2 with erfc from Abramowitz & Stegun, Handbook of Mathematical Functions, 7.1.26 (absolute error
+// 1.5e-7): erfc(x) = (a1 t + .. + a5 t^5) exp(-x^2), t = 1 / (1 + p x), x >= 0.  No branch, and a negative z multiplies erfc itself, so its
+// small values keep their relative accuracy; the value is rounded to bf16 right after
+__device__ __forceinline__ float sq_gelu_erf(float z) {
+    const float x = fabsf(z) * 0.70710678118654752f;
+    const float t = __fdividef(1.0f, fmaf(0.3275911f, x, 1.0f));
+    float q = fmaf(t, 1.061405429f, -1.453152027f);
+    q = fmaf(t, q, 1.421413741f);
+    q = fmaf(t, q, -0.284496736f);
+    q = fmaf(t, q, 0.254829592f);
+    q *= t * __expf(-x * x);
+    return 0.5f * z * (z < 0.0f ? q : 2.0f - q);
+}
 __device__ __forceinline__ float sq_gate(float z, int kind) { return kind ? sq_silu(z) : sq_gelu(z); }
 
 template <int BN, int EPI>
@@ -199,8 +213,13 @@ k_seq_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUte
                         }
                     }
                 }
-            } else if (EPI == SQ_EPI_RELU2) {
-                const float wt = row < M ? ep.row_w[row] : 0.0f;
+            } else if (EPI == SQ_EPI_RELU2 || EPI == SQ_EPI_GELU) {
+                const float wt = (EPI == SQ_EPI_RELU2 && row < M) ? ep.row_w[row] : 0.0f;
+                auto act = [wt](float a) {
+                    if (EPI == SQ_EPI_GELU) return sq_gelu_erf(a);
+                    a = fmaxf(a, 0.0f);
+                    return wt * a * a;
+                };
 #pragma unroll 1
                 for (int c = chalf * (BN / 64); c < (chalf + 1) * (BN / 64); c++) {
                     const int col = nt * BN + c * 32;
@@ -215,8 +234,7 @@ k_seq_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUte
                                 uint32_t w[4];
 #pragma unroll
                                 for (int q = 0; q < 4; q++) {
-                                    const float a0 = fmaxf(v[j + 2 * q], 0.0f), a1 = fmaxf(v[j + 2 * q + 1], 0.0f);
-                                    const __nv_bfloat162 pr = __floats2bfloat162_rn(wt * a0 * a0, wt * a1 * a1);
+                                    const __nv_bfloat162 pr = __floats2bfloat162_rn(act(v[j + 2 * q]), act(v[j + 2 * q + 1]));
                                     w[q] = *reinterpret_cast<const uint32_t*>(&pr);
                                 }
                                 *reinterpret_cast<uint4*>(dst + j) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -224,7 +242,7 @@ k_seq_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUte
                         } else {
 #pragma unroll
                             for (int j = 0; j < 32; j++)
-                                if (j < nc) { const float a0 = fmaxf(v[j], 0.0f); dst[j] = __float2bfloat16_rn(wt * a0 * a0); }
+                                if (j < nc) dst[j] = __float2bfloat16_rn(act(v[j]));
                         }
                     }
                 }
@@ -279,7 +297,7 @@ typedef CUresult (*PFN_tmapEncodeTiled)(CUtensorMap*, CUtensorMapDataType, cuuin
 struct SeqGemmPlan {
     PFN_tmapEncodeTiled enc = nullptr;
     int* d_status = nullptr;
-    bool attr[2][3] = {{false, false, false}, {false, false, false}};
+    bool attr[2][4] = {{false, false, false, false}, {false, false, false, false}};
 };
 
 int seq_gemm_create(SeqGemmPlan** out) {
@@ -346,6 +364,7 @@ static int run(SeqGemmPlan* p, int epi, const void* A, int lda, const void* W, i
     if (rc) return rc;
     rc = make_map(p, &tb, W, N, K, ldw, bn);
     if (rc) return rc;
+    if (epi == SQ_EPI_GELU) return bn == 256 ? launch<256, SQ_EPI_GELU>(p, ta, tb, M, N, K, ep) : launch<128, SQ_EPI_GELU>(p, ta, tb, M, N, K, ep);
     if (epi == SQ_EPI_F32) return bn == 256 ? launch<256, SQ_EPI_F32>(p, ta, tb, M, N, K, ep) : launch<128, SQ_EPI_F32>(p, ta, tb, M, N, K, ep);
     return bn == 256 ? launch<256, SQ_EPI_GEGLU>(p, ta, tb, M, N, K, ep) : launch<128, SQ_EPI_GEGLU>(p, ta, tb, M, N, K, ep);
 }
@@ -354,6 +373,12 @@ int seq_gemm_bf16(SeqGemmPlan* p, const void* A, int lda, const void* W, int ldw
     SqEpi ep{};
     ep.C = C; ep.ldc = ldc; ep.bias = bias; ep.accumulate = accumulate; ep.status = p ? p->d_status : nullptr;
     return run(p, SQ_EPI_F32, A, lda, W, ldw, M, N, K, ep);
+}
+
+int seq_gemm_bf16_gelu(SeqGemmPlan* p, const void* A, int lda, const void* W, int ldw, void* act, int ld_act, int M, int N, int K) {
+    SqEpi ep{};
+    ep.act = reinterpret_cast<__nv_bfloat16*>(act); ep.ld_act = ld_act; ep.status = p ? p->d_status : nullptr;
+    return run(p, SQ_EPI_GELU, A, lda, W, ldw, M, N, K, ep);
 }
 
 int seq_gemm_bf16_grouped(SeqGemmPlan* p, const void* A, int lda, const void* W, int ldw, int M_pad, int N, int K, int n_groups, const int* tile_group,

@@ -18,6 +18,8 @@ int seq_gemm_bf16_geglu(SeqGemmPlan* p, const void* A, int lda, const void* W, i
 // the same with a choice of activation (act_kind 0: gelu_tanh(gate) * up, 1: silu(gate) * up) and an optional weight per row of A
 int seq_gemm_bf16_gated(SeqGemmPlan* p, const void* A, int lda, const void* W, int ldw, void* act, int ld_act, int act_off, int M, int N2, int K, int act_kind,
                         const float* row_w);
+// ungated feed-forward input: act[row][c] = bf16(gelu(A . W^T)) for c < N, gelu in its erf form
+int seq_gemm_bf16_gelu(SeqGemmPlan* p, const void* A, int lda, const void* W, int ldw, void* act, int ld_act, int M, int N, int K);
 // grouped and gated: group g multiplies with rows [g N2, (g + 1) N2) of W (its gate and up rows interleaved in groups of 32);
 // act[row][c] = bf16(row_w[row] * act(gate_c) * up_c) for c < N2 / 2
 int seq_gemm_bf16_grouped_gated(SeqGemmPlan* p, const void* A, int lda, const void* W, int ldw, int M_pad, int N2, int K, int n_groups, const int* tile_group,

@@ -227,7 +227,7 @@ __global__ void k_copy_operand(const float* __restrict__ h, int width, OT* __res
 }
 // history <- the last taps - 1 values of h of each segment's sequence.  One thread per channel walks k upwards: entry k is written
 // after every entry it is read for (k + len > k).
-__global__ void k_canon_tail(PassTables t, const float* __restrict__ h, int width, int taps, float* __restrict__ tail) {
+__global__ void k_canon_tail(PassTables t, const float* __restrict__ h, int ldh, int width, int taps, float* __restrict__ tail) {
     const int s = blockIdx.x;
     const int row0 = t.seg_row0[s], len = t.seg_len[s], slot = t.seg_slot[s];
     if (t.slots[slot].stopped) return;
@@ -235,7 +235,7 @@ __global__ void k_canon_tail(PassTables t, const float* __restrict__ h, int widt
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < width; c += gridDim.y * blockDim.x)
         for (int k = 0; k < taps - 1; k++) {
             const int off = len - (taps - 1) + k;          // offset inside the segment of the row that lands in entry k
-            tl[(size_t)k * width + c] = (off >= 0) ? h[(size_t)(row0 + off) * width + c] : tl[(size_t)(k + len) * width + c];
+            tl[(size_t)k * width + c] = (off >= 0) ? h[(size_t)(row0 + off) * ldh + c] : tl[(size_t)(k + len) * width + c];
         }
 }
 

@@ -148,9 +148,12 @@ __global__ void __launch_bounds__(256) k_dyt_rows(const float* __restrict__ x, i
         out[(size_t)o * ld_out + c] = cvt<OUT>(fmaf(tanhf(a * x[(size_t)r * width + c]), nrm.w[c], nrm.b[c]));
 }
 
-__global__ void k_softcap(float* __restrict__ v, size_t n, float cap) {
+// logits <- scale * logits, then cap * tanh(. / cap) when cap > 0
+__global__ void k_logits_post(float* __restrict__ v, size_t n, float scale, float cap) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) v[i] = cap * tanhf(v[i] / cap);
+    if (i >= n) return;
+    const float z = scale * v[i];
+    v[i] = cap > 0.0f ? cap * tanhf(z / cap) : z;
 }
 
 // ------------------------------------------------------------------------------------------------ latent attention
@@ -162,6 +165,8 @@ struct LatAttn {
     float eps;
     int q_off, kv_off, g_off;    // columns of [q | dq], dkv and the gates in the projection buffer
     int a_off;
+    float rot_amp;               // factor on cos and sin of the rotation (frequency scaling), 1 without
+    int own_kv;                  // 0: latents and rotated key parts are another layer's cache (nothing is projected or appended here)
     int c_ld;                    // row stride of the latent cache [n_slots][max_ctx][c_ld]: latent, then the rotated key part
     int max_ctx;
 };
@@ -170,8 +175,9 @@ __device__ __forceinline__ void rot_pair(const LatAttn& b, int pr, int& i0, int&
     i1 = b.rot_layout ? 2 * pr + 1 : pr + b.rot_dims / 2;
 }
 
-// per row: latent = unit-RMS(dkv[:rank]) * kv_norm and the rotated key part -> the slot's cache row (CTA y = 0); with a query latent,
-// unit-RMS(dq) * q_norm -> the operand of the query up-projection, zero-padded to ld_q (CTA y = 1)
+// per row: latent = unit-RMS(dkv[:rank]) * kv_norm and the rotated key part -> the slot's cache row; with a query latent,
+// unit-RMS(dq) * q_norm -> the operand of the query up-projection, zero-padded to ld_q.  grid (rows, parts): the parts are [cache row, if the
+// layer has its own] [query latent, if there is one]
 template <typename OT>
 __global__ void __launch_bounds__(128) k_lat_prep(PassTables t, LatAttn b, const float* __restrict__ P, int ldp, OT* __restrict__ cache,
                                                   OT* __restrict__ opq, int ld_q) {
@@ -179,7 +185,7 @@ __global__ void __launch_bounds__(128) k_lat_prep(PassTables t, LatAttn b, const
     const int r = blockIdx.x;
     const int slot = t.seg_slot[t.row_seg[r]], pos = t.row_pos[r];
     const float* p = P + (size_t)r * ldp;
-    if (blockIdx.y == 1) {                               // the query latent (grid y = 2 only with one)
+    if (blockIdx.y == 1 || !b.own_kv) {                  // the query latent
         float sq_ = 0.0f;
         for (int i = threadIdx.x; i < b.q_rank; i += blockDim.x) { const float v = p[b.q_off + i]; sq_ += v * v; }
         sq_ = block_sum(sq_, red);
@@ -200,16 +206,16 @@ __global__ void __launch_bounds__(128) k_lat_prep(PassTables t, LatAttn b, const
         rot_pair(b, pr, i0, i1);
         float sn, cs;
         sincosf(fpos * b.inv_freq[pr], &sn, &cs);
+        sn *= b.rot_amp; cs *= b.rot_amp;
         dst[b.rank + i0] = cvt<OT>(kr[i0] * cs - kr[i1] * sn);
         dst[b.rank + i1] = cvt<OT>(kr[i1] * cs + kr[i0] * sn);
     }
     for (int i = b.rot_dims + threadIdx.x; i < b.rope; i += blockDim.x) dst[b.rank + i] = cvt<OT>(kr[i]);
 }
 
-// Prompt portions: the heads' queries with their rotated part turned to the row's position, and the heads' gate logits behind them:
-// QR [R][ld_qr] = [heads x (plain | rotated) | heads gates].  Q may be QR itself (in place).
-__global__ void __launch_bounds__(128) k_lat_qrot(PassTables t, LatAttn b, const float* __restrict__ Q, int ldq, int q0, const float* __restrict__ P, int ldp,
-                                                  float* __restrict__ QR, int ld_qr) {
+// Prompt portions: the heads' queries with their rotated part turned to the row's position: QR [R][ld_qr] = heads x (plain | rotated).
+// Q may be QR itself (in place).
+__global__ void __launch_bounds__(128) k_lat_qrot(PassTables t, LatAttn b, const float* Q, int ldq, int q0, float* QR, int ld_qr) {
     const int r = blockIdx.x, hd = b.dim + b.rope;
     const float fpos = (float)t.row_pos[r];
     const float* q = Q + (size_t)r * ldq + q0;
@@ -225,11 +231,11 @@ __global__ void __launch_bounds__(128) k_lat_qrot(PassTables t, LatAttn b, const
         rot_pair(b, pr, i0, i1);
         float sn, cs;
         sincosf(fpos * b.inv_freq[pr], &sn, &cs);
+        sn *= b.rot_amp; cs *= b.rot_amp;
         const float u = q[h * hd + b.dim + i0], v = q[h * hd + b.dim + i1];
         o[h * hd + b.dim + i0] = u * cs - v * sn;
         o[h * hd + b.dim + i1] = v * cs + u * sn;
     }
-    if (P) for (int h = threadIdx.x; h < b.heads; h += blockDim.x) o[b.heads * hd + h] = P[(size_t)r * ldp + b.g_off + h];
 }
 
 // Expanded keys and values of n cached tokens of one slot from position lo: X [n][heads * (dim + vdim)] (fp32) holds [uk c | uv c];
@@ -294,6 +300,7 @@ __global__ void __launch_bounds__(128) k_lat_qabs(PassTables t, LatAttn b, const
         rot_pair(b, pr, i0, i1);
         float sn, cs;
         sincosf(fpos * b.inv_freq[pr], &sn, &cs);
+        sn *= b.rot_amp; cs *= b.rot_amp;
         qa[b.rank + i0] = qr[i0] * cs - qr[i1] * sn;
         qa[b.rank + i1] = qr[i1] * cs + qr[i0] * sn;
     }
@@ -459,8 +466,9 @@ __global__ void __launch_bounds__(128) k_lat_dec_mma(PassTables t, SoftAttn b, c
         }
 }
 
-// Value up-projection of the summed latents and the head's gate: out[r][a_off + h vdim + v] = logistic(P[r][g_off + h]) * uv[h vdim + v] . ol[r][h]
-// OL [R][ld_ol] holds heads x rank summed latents; a warp per output entry.  gate 0: no gate.
+// Value up-projection of the summed latents and the gate: out[r][a_off + h vdim + v] = logistic(P[r][g_off + h]) * uv[h vdim + v] . ol[r][h]
+// OL [R][ld_ol] holds heads x rank summed latents; a warp per output entry.  gate 0: no gate; 2: one gate per entry (column g_off + h vdim + v)
+// instead of one per head.
 template <typename OT>
 __global__ void __launch_bounds__(256) k_lat_vup(LatAttn b, const OT* __restrict__ OL, int ld_ol, const bf16* __restrict__ uv, int ld_uv,
                                                  const float* __restrict__ P, int ldp, int gate, OT* __restrict__ out, int ld_out) {
@@ -489,7 +497,7 @@ __global__ void __launch_bounds__(256) k_lat_vup(LatAttn b, const OT* __restrict
         }
         s = warp_sum(s);
         if (lane == 0) {
-            if (gate) s *= sigmoidf_(P[(size_t)r * ldp + b.g_off + h]);
+            if (gate) s *= sigmoidf_(P[(size_t)r * ldp + b.g_off + (gate == 2 ? e : h)]);
             out[(size_t)r * ld_out + b.a_off + e] = cvt<OT>(s);
         }
     }

@@ -339,7 +339,19 @@ struct SoftAttn {
     int chunk;                   // > 0: a query sees only keys of its own chunk of positions
     float out_scale;             // weight of the output (0 counts as 1)
     const float* qk_sc;          // qk_norm 3
+    float rot_amp;               // factor on cos and sin of the rotation (frequency scaling), 1 without
+    int keep;                    // > 0: the first `keep` tokens stay visible outside the window or chunk (not with pool)
+    const float* slope;          // [heads] or null: slope[head] * (query position - key position) is taken off the score (not with pool)
+    int v_is_k;                  // the value cache IS the key cache (dim = vdim, same heads)
+    const float* gate_src;       // [rows][gate_ld]: where gate logits are read (column g_off ..); null: the buffer the queries come from
+    int gate_ld;
 };
+// gate factor of (row, query unit h, channel c) of head hd
+__device__ __forceinline__ float sa_gate(const SoftAttn& b, const float* __restrict__ P, int ldp, int r, int hd, int h, int c) {
+    const float* g = b.gate_src ? b.gate_src + (size_t)r * b.gate_ld : P + (size_t)r * ldp;
+    const float gt = g[b.g_off + (b.gate == 3 ? hd : h * b.vdim + c)];
+    return b.gate >= 2 ? sigmoidf_(gt) : gt * sigmoidf_(gt);
+}
 __host__ __device__ __forceinline__ int sa_maps(const SoftAttn& b) { return b.maps > 1 ? b.maps : 1; }
 
 // q (and k): per-head norm, rotary positions; q in place (fp32), k and v appended to the slot's cache.
@@ -371,6 +383,7 @@ __global__ void __launch_bounds__(128) k_sattn_prep(PassTables t, SoftAttn b, fl
                 const float a = v[i0] * sc * (wn ? wn[i0] : 1.0f), c = v[i1] * sc * (wn ? wn[i1] : 1.0f);
                 float sn, cs;
                 sincosf(fpos * b.inv_freq[pr], &sn, &cs);
+                sn *= b.rot_amp; cs *= b.rot_amp;
                 const float ra = a * cs - c * sn, rc = c * cs + a * sn;
                 if (is_q) { v[i0] = ra; v[i1] = rc; } else { dst[i0] = cvt<OT>(ra); dst[i1] = cvt<OT>(rc); }
             }
@@ -424,14 +437,16 @@ __global__ void __launch_bounds__(128) k_pool_update(PassTables t, SoftAttn b, c
 }
 
 __device__ __forceinline__ float soft_cap(float s, float cap) { return cap > 0.0f ? cap * tanhf(s / cap) : s; }
-// keys a query at `pos` sees: pooled blocks 0 .. nb-1 (those that end at or before pos - window), then tokens lo .. pos
+// keys a query at `pos` sees: tokens lo .. pos and, in front of them in the key list, nb others: pooled blocks 0 .. nb-1 (those that end at
+// or before pos - window), or the kept first tokens 0 .. nb-1 that lie before lo
 __device__ __forceinline__ void sattn_range(const SoftAttn& b, int pos, int& lo, int& nb) {
     lo = b.window > 0 ? max(0, pos - b.window + 1) : 0;
     if (b.chunk > 0) lo = max(lo, pos / b.chunk * b.chunk);
     nb = (b.window > 0 && b.pool > 0 && pos - b.window + 1 >= b.pool) ? (pos - b.window + 1) / b.pool : 0;
+    if (b.keep > 0) nb = min(b.keep, lo);
 }
 
-// Online softmax of one (row, query head) over the keys n_lo .. n_hi-1 of the list [pooled blocks | window tokens], in tiles of
+// Online softmax of one (row, query head) over the keys n_lo .. n_hi-1 of the list [pooled blocks or kept tokens | window tokens], in tiles of
 // blockDim.x keys: a thread scores one key of the tile, then the threads turn to the value channels (vdim <= 4 * blockDim.x).
 // m, l: running maximum and denominator (in / out); acc: this thread's value channels.  sm: dim + blockDim.x + 33 floats.
 template <typename OT>
@@ -449,14 +464,17 @@ __device__ __forceinline__ void sattn_sweep(const PassTables& t, const SoftAttn&
     const OT* vbase = vc + (size_t)slot * b.max_ctx * vld + (size_t)g * b.vdim;
     const float* pkb = pk ? pk + (size_t)slot * b.max_blocks * kld + (size_t)ku * b.dim : nullptr;
     const float* pvb = pv ? pv + (size_t)slot * b.max_blocks * vld + (size_t)g * b.vdim : nullptr;
-    const bool kvec = b.dim % 8 == 0 && kld % 8 == 0;
+    const bool kvec = b.dim % 8 == 0 && kld % 8 == 0, pooled = b.keep <= 0;
+    const float slope = b.slope ? b.slope[h / M] : 0.0f;
+    const int pos = t.row_pos[r];
     __syncthreads();
     for (int n0 = n_lo; n0 < n_hi; n0 += blockDim.x) {
         const int n = n0 + threadIdx.x;
         float s = -INFINITY;
         if (n < n_hi) {
-            const float d = n < nb ? key_dot(sq, pkb + (size_t)n * kld, b.dim, b.dim % 4 == 0) : key_dot(sq, kbase + (size_t)(lo + n - nb) * kld, b.dim, kvec);
-            s = soft_cap(d * b.scale, b.softcap);
+            const int j = n < nb ? n : lo + n - nb;
+            const float d = n < nb && pooled ? key_dot(sq, pkb + (size_t)n * kld, b.dim, b.dim % 4 == 0) : key_dot(sq, kbase + (size_t)j * kld, b.dim, kvec);
+            s = soft_cap(d * b.scale, b.softcap) - slope * (float)(pos - j);
         }
         const float mn = fmaxf(m, block_max(s, red));
         const float corr = m == -INFINITY ? 0.0f : expf(m - mn);
@@ -472,7 +490,7 @@ __device__ __forceinline__ void sattn_sweep(const PassTables& t, const SoftAttn&
                 float a = acc[cc] * corr;
                 for (int jj = 0; jj < nj; jj++) {
                     const int nn = n0 + jj;
-                    const float v = nn < nb ? pvb[(size_t)nn * vld + c] : ldf<OT>(vbase + (size_t)(lo + nn - nb) * vld + c);
+                    const float v = nn < nb && pooled ? pvb[(size_t)nn * vld + c] : ldf<OT>(vbase + (size_t)(nn < nb ? nn : lo + nn - nb) * vld + c);
                     a = fmaf(swt[jj], v, a);
                 }
                 acc[cc] = a;
@@ -490,10 +508,7 @@ __device__ __forceinline__ void sattn_store(const SoftAttn& b, const float* __re
         const int c = threadIdx.x + cc * blockDim.x;
         if (c < b.vdim) {
             float o = acc[cc] * inv;
-            if (b.gate) {
-                const float gt = P[(size_t)r * ldp + b.g_off + (b.gate == 3 ? h / sa_maps(b) : h * b.vdim + c)];
-                o *= b.gate >= 2 ? sigmoidf_(gt) : gt * sigmoidf_(gt);
-            }
+            if (b.gate) o *= sa_gate(b, P, ldp, r, h / sa_maps(b), h, c);
             out[(size_t)r * ld_out + b.a_off + h * b.vdim + c] = cvt<OT>(o);
         }
     }

@@ -14,9 +14,9 @@ __device__ __forceinline__ float sa_tanh(float z) {
 }
 
 // A CTA owns 64 consecutive rows of one segment and one query head (4 warps x 16 rows).  It sweeps, in tiles of 64 keys, first the
-// pooled blocks that its last row sees (fp32 means converted to bf16 on the way into shared memory), then the tokens from the first
-// row's window start to the last row: S = Q K^T, score = cap(scale S) under the row's own mask (block b: (b + 1) pool <= pos - window + 1;
-// token j: pos - window < j <= pos), online softmax in fp32 whose running maximum starts at the sink (so the sink's term is
+// pooled blocks that its last row sees (fp32 means converted to bf16 on the way into shared memory) or the kept first tokens, then the
+// tokens from the first row's window start to the last row: S = Q K^T, score = cap(scale S) - slope (pos - j) under the row's own mask
+// (block b: (b + 1) pool <= pos - window + 1; kept token j < keep before the row's window; token j: pos - window < j <= pos), online softmax in fp32 whose running maximum starts at the sink (so the sink's term is
 // exp(sink - max) at the end and counts once), O += P V with P as bf16 A fragments straight from the accumulator registers.
 // Soft-capping uses the special-function tanh (relative error 2^-11, below the bf16 rounding of the weights that follow).
 template <int DP, int VP>
@@ -44,16 +44,18 @@ __global__ void __launch_bounds__(128) k_sattn_mma(PassTables t, SoftAttn b, int
     const float* pkb = pk ? pk + (size_t)slot * b.max_blocks * kld + (size_t)ku * b.dim : nullptr;
     const float* pvb = pv ? pv + (size_t)slot * b.max_blocks * vld + (size_t)g * b.vdim : nullptr;
     const bool vec = (b.dim % 8 == 0) && (b.vdim % 8 == 0);
+    const bool one_tile = b.v_is_k && DP == VP;          // keys double as values: one tile in shared memory serves both products
+    const bool pooled = b.keep <= 0;
     const int last = pos0 + nq - 1;                      // last position of the tile
     int t_lo, nb_tile;
-    sattn_range(b, last, t_lo, nb_tile);                 // blocks the last row sees: the most of any row
+    sattn_range(b, last, t_lo, nb_tile);                 // blocks / kept tokens the last row sees: the most of any row
     { int nb0; sattn_range(b, pos0, t_lo, nb0); }     // the first row's first token: the lowest of any row
     const int n_bt = (nb_tile + 63) / 64, n_it = n_bt + (last - t_lo) / 64 + 1;
     const uint32_t sq_a = (uint32_t)__cvta_generic_to_shared(sq);
     auto load_tile = [&](int st, int it) {
         bf16* sk = sk0 + st * 64 * LQ;
         bf16* sv = sv0 + st * 64 * LV;
-        if (it < n_bt) {
+        if (it < n_bt && pooled) {
             const int b0 = it * 64, nk = min(64, nb_tile - b0);
             for (int e = threadIdx.x; e < 64 * DP; e += 128) {
                 const int r = e / DP, i = e % DP;
@@ -64,7 +66,8 @@ __global__ void __launch_bounds__(128) k_sattn_mma(PassTables t, SoftAttn b, int
                 sv[r * LV + i] = __float2bfloat16_rn((r < nk && i < b.vdim) ? pvb[(size_t)(b0 + r) * vld + i] : 0.0f);
             }
         } else {
-            const int j0 = t_lo + (it - n_bt) * 64, nk = min(64, last + 1 - j0);
+            const bool kept = it < n_bt;
+            const int j0 = kept ? it * 64 : t_lo + (it - n_bt) * 64, nk = min(64, (kept ? nb_tile : last + 1) - j0);
             if (vec) {
                 const uint32_t ka = (uint32_t)__cvta_generic_to_shared(sk), va = (uint32_t)__cvta_generic_to_shared(sv);
                 for (int e = threadIdx.x; e < 64 * (DP / 8); e += 128) {
@@ -72,7 +75,7 @@ __global__ void __launch_bounds__(128) k_sattn_mma(PassTables t, SoftAttn b, int
                     const bool ok = r < nk && c8 < b.dim;
                     sa_cp16(ka + (uint32_t)((r * LQ + c8) * 2), ok ? (const void*)(kbase + (size_t)(j0 + r) * kld + c8) : (const void*)kbase, ok);
                 }
-                for (int e = threadIdx.x; e < 64 * (VP / 8); e += 128) {
+                if (!one_tile) for (int e = threadIdx.x; e < 64 * (VP / 8); e += 128) {
                     const int r = e / (VP / 8), c8 = (e % (VP / 8)) * 8;
                     const bool ok = r < nk && c8 < b.vdim;
                     sa_cp16(va + (uint32_t)((r * LV + c8) * 2), ok ? (const void*)(vbase + (size_t)(j0 + r) * vld + c8) : (const void*)vbase, ok);
@@ -82,7 +85,7 @@ __global__ void __launch_bounds__(128) k_sattn_mma(PassTables t, SoftAttn b, int
                     const int r = e / DP, i = e % DP;
                     sk[r * LQ + i] = (r < nk && i < b.dim) ? kbase[(size_t)(j0 + r) * kld + i] : __float2bfloat16_rn(0.0f);
                 }
-                for (int e = threadIdx.x; e < 64 * VP; e += 128) {
+                if (!one_tile) for (int e = threadIdx.x; e < 64 * VP; e += 128) {
                     const int r = e / VP, i = e % VP;
                     sv[r * LV + i] = (r < nk && i < b.vdim) ? vbase[(size_t)(j0 + r) * vld + i] : __float2bfloat16_rn(0.0f);
                 }
@@ -104,7 +107,7 @@ __global__ void __launch_bounds__(128) k_sattn_mma(PassTables t, SoftAttn b, int
     float o[VP / 8][4];
 #pragma unroll
     for (int n = 0; n < VP / 8; n++) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f; }
-    const float inv_cap = b.softcap > 0.0f ? 1.0f / b.softcap : 0.0f;
+    const float inv_cap = b.softcap > 0.0f ? 1.0f / b.softcap : 0.0f, slope = b.slope ? b.slope[hd] : 0.0f;
     load_tile(0, 0);
     for (int it = 0; it < n_it; it++) {
         const int st = it & 1;
@@ -114,10 +117,10 @@ __global__ void __launch_bounds__(128) k_sattn_mma(PassTables t, SoftAttn b, int
         else asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         const bool is_blk = it < n_bt;
-        const int k0 = is_blk ? it * 64 : t_lo + (it - n_bt) * 64;
+        const int k0 = is_blk ? it * 64 : t_lo + (it - n_bt) * 64;       // first key of the tile: a block's number, or a token's position
         const bool skip = is_blk ? (k0 >= nb_w) : (k0 > pw1 || k0 + 63 < wl0);
         if (skip) { __syncthreads(); continue; }        // no row of this warp sees a key of the tile
-        const uint32_t sk_a = (uint32_t)__cvta_generic_to_shared(sk0 + st * 64 * LQ), sv_a = (uint32_t)__cvta_generic_to_shared(sv0 + st * 64 * LV);
+        const uint32_t sk_a = (uint32_t)__cvta_generic_to_shared(sk0 + st * 64 * LQ), sv_a = one_tile ? sk_a : (uint32_t)__cvta_generic_to_shared(sv0 + st * 64 * LV);
         float sc[8][4];
 #pragma unroll
         for (int n = 0; n < 8; n++) { sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.0f; }
@@ -144,6 +147,7 @@ __global__ void __launch_bounds__(128) k_sattn_mma(PassTables t, SoftAttn b, int
                 const bool vis = is_blk ? key < (hi ? nb_hi : nb_lo) : (key <= (hi ? p_hi : p_lo) && key >= (hi ? tl_hi : tl_lo));
                 float s = sc[n][x] * b.scale;
                 if (b.softcap > 0.0f) s = b.softcap * sa_tanh(s * inv_cap);
+                if (b.slope) s -= slope * (float)((hi ? p_hi : p_lo) - key);
                 s = vis ? s : -INFINITY;
                 sc[n][x] = s;
                 if (hi) mx_hi = fmaxf(mx_hi, s); else mx_lo = fmaxf(mx_lo, s);
@@ -206,12 +210,12 @@ __global__ void __launch_bounds__(128) k_sattn_mma(PassTables t, SoftAttn b, int
             if (c + x >= b.vdim) continue;
             if (r_lo < nq) {
                 float v = o[n][x] * i_lo * os;
-                if (b.gate) { const float gt = P[(size_t)(row0 + r_lo) * ldp + b.g_off + (b.gate == 3 ? hd : h * b.vdim + c + x)]; v *= b.gate >= 2 ? sigmoidf_(gt) : gt * sigmoidf_(gt); }
+                if (b.gate) v *= sa_gate(b, P, ldp, row0 + r_lo, hd, h, c + x);
                 out[(size_t)(row0 + r_lo) * ld_out + b.a_off + h * b.vdim + c + x] = __float2bfloat16_rn(v);
             }
             if (r_hi < nq) {
                 float v = o[n][2 + x] * i_hi * os;
-                if (b.gate) { const float gt = P[(size_t)(row0 + r_hi) * ldp + b.g_off + (b.gate == 3 ? hd : h * b.vdim + c + x)]; v *= b.gate >= 2 ? sigmoidf_(gt) : gt * sigmoidf_(gt); }
+                if (b.gate) v *= sa_gate(b, P, ldp, row0 + r_hi, hd, h, c + x);
                 out[(size_t)(row0 + r_hi) * ld_out + b.a_off + h * b.vdim + c + x] = __float2bfloat16_rn(v);
             }
         }

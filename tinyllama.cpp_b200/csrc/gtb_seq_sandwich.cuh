@@ -6,6 +6,8 @@
 //   * differential attention: the combination of a head's two score maps, its unit-RMS norm and gate
 //   * retention with SiLU-activated inputs, an RMS norm over the concatenated heads and a logistic gate
 //   * a sigmoid router whose choice is limited to the best groups of experts
+//   * a short causal convolution right behind the query and key projections, with the cache append behind it
+//   * the erf form of GELU as the activation of an ungated feed-forward
 // The attention and retention kernels themselves are those of gtb_seq_mixers*.cuh and gtb_seq_kernels.cuh.
 //
 // Precision follows gtb_seq_kernels.cuh: everything below is fp32 except operands of matrix products (type OT).
@@ -15,7 +17,7 @@
 namespace gtb {
 namespace seq {
 
-constexpr int SW_NORM_LAYER = 2;            // NormArgs::kind of a layer norm (GTB_NORM_LAYER); anything else here: RMS with a plain weight
+constexpr int SW_NORM_LAYER = 2;            // NormArgs::kind of a layer norm (GTB_NORM_LAYER); anything else here: RMS with a plain weight.  b null: no bias
 
 // Sum over the block with ONE barrier: every warp leaves its partial sum in `slot` (32 floats that no other reduction of the kernel uses, so
 // nothing has to wait for earlier readers) and every thread adds the partial sums itself, in the same order.
@@ -51,9 +53,10 @@ __device__ __forceinline__ void sw_stats(const float (&v)[4 * N4], int width, in
     rstd = 1.0f / sqrtf(sw_block_sum(ss, red + 32) / (float)width + eps);
 }
 
-// out = norm(x[rows[o]]) as a product operand.  rows: optional gather.
+// out = out_scale * norm(x[rows[o]]) as a product operand.  rows: optional gather.
 template <typename OT>
-__global__ void __launch_bounds__(256) k_norm_rows(const float* __restrict__ x, int width, NormArgs nrm, const int* __restrict__ rows, OT* __restrict__ out, int ld_out) {
+__global__ void __launch_bounds__(256) k_norm_rows(const float* __restrict__ x, int width, NormArgs nrm, const int* __restrict__ rows, OT* __restrict__ out, int ld_out,
+                                                   float out_scale) {
     __shared__ float red[33];
     const int o = blockIdx.x, r = rows ? rows[o] : o, center = nrm.kind == SW_NORM_LAYER;
     const float* xr = x + (size_t)r * width;
@@ -67,7 +70,7 @@ __global__ void __launch_bounds__(256) k_norm_rows(const float* __restrict__ x, 
     for (int c = threadIdx.x; c < width; c += blockDim.x) { const float d = xr[c] - mean; ss += d * d; }
     const float rstd = 1.0f / sqrtf(block_sum(ss, red) / (float)width + nrm.eps);
     for (int c = threadIdx.x; c < width; c += blockDim.x)
-        out[(size_t)o * ld_out + c] = cvt<OT>((xr[c] - mean) * rstd * nrm.w[c] + (center ? nrm.b[c] : 0.0f));
+        out[(size_t)o * ld_out + c] = cvt<OT>(((xr[c] - mean) * rstd * nrm.w[c] + (nrm.b ? nrm.b[c] : 0.0f)) * out_scale);
 }
 
 // ------------------------------------------------------------------------------------------------ group-limited sigmoid router
@@ -181,7 +184,7 @@ __global__ void __launch_bounds__(256) k_embed_norm(PassTables t, const bf16* __
     float ss = 0.0f;
     for (int c = threadIdx.x; c < width; c += blockDim.x) { const float d = xr[c] - mean; ss += d * d; }      // a thread re-reads what it wrote
     const float rstd = 1.0f / sqrtf(block_sum(ss, red) / (float)width + nrm.eps);
-    for (int c = threadIdx.x; c < width; c += blockDim.x) op[(size_t)r * ld_op + c] = cvt<OT>((xr[c] - mean) * rstd * nrm.w[c] + (center ? nrm.b[c] : 0.0f));
+    for (int c = threadIdx.x; c < width; c += blockDim.x) op[(size_t)r * ld_op + c] = cvt<OT>((xr[c] - mean) * rstd * nrm.w[c] + (nrm.b ? nrm.b[c] : 0.0f));
 }
 
 // Residual update of the sandwich style: y = Y (+ Y2), or the sum of rows pair_dst[r * top + k] >= 0 of Yg (grouped experts, in order of k);
@@ -227,7 +230,7 @@ __global__ void __launch_bounds__(256, SW_KEEP == 4 ? 4 : SW_KEEP == 2 ? 6 : 8) 
             const int c = (threadIdx.x + i * blockDim.x) * 4;
             if (c < width) {
                 const float4 w4 = *reinterpret_cast<const float4*>(post.w + c);
-                const float4 b4 = cp ? *reinterpret_cast<const float4*>(post.b + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                const float4 b4 = post.b ? *reinterpret_cast<const float4*>(post.b + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
                 vx[4 * i] += (vy[4 * i] - mean) * rstd * w4.x + b4.x; vx[4 * i + 1] += (vy[4 * i + 1] - mean) * rstd * w4.y + b4.y;
                 vx[4 * i + 2] += (vy[4 * i + 2] - mean) * rstd * w4.z + b4.z; vx[4 * i + 3] += (vy[4 * i + 3] - mean) * rstd * w4.w + b4.w;
                 *reinterpret_cast<float4*>(xr + c) = make_float4(vx[4 * i], vx[4 * i + 1], vx[4 * i + 2], vx[4 * i + 3]);
@@ -240,7 +243,7 @@ __global__ void __launch_bounds__(256, SW_KEEP == 4 ? 4 : SW_KEEP == 2 ? 6 : 8) 
             const int c = (threadIdx.x + i * blockDim.x) * 4;
             if (c < width) {
                 const float4 w4 = *reinterpret_cast<const float4*>(next.w + c);
-                const float4 b4 = cn ? *reinterpret_cast<const float4*>(next.b + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                const float4 b4 = next.b ? *reinterpret_cast<const float4*>(next.b + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
                 const float h0 = (vx[4 * i] - mean) * rstd * w4.x + b4.x, h1 = (vx[4 * i + 1] - mean) * rstd * w4.y + b4.y;
                 const float h2 = (vx[4 * i + 2] - mean) * rstd * w4.z + b4.z, h3 = (vx[4 * i + 3] - mean) * rstd * w4.w + b4.w;
                 store4(op + (size_t)r * ld_op + c, h0, h1, h2, h3);
@@ -267,7 +270,7 @@ __global__ void __launch_bounds__(256, SW_KEEP == 4 ? 4 : SW_KEEP == 2 ? 6 : 8) 
     s = 0.0f;
     for (int c = threadIdx.x; c < width; c += blockDim.x) { const float d = sub(c) - mean; s += d * d; }
     float rstd = 1.0f / sqrtf(block_sum(s, red) / (float)width + post.eps);
-    for (int c = threadIdx.x; c < width; c += blockDim.x) xr[c] += (sub(c) - mean) * rstd * post.w[c] + (cp ? post.b[c] : 0.0f);     // a thread re-reads only what it wrote
+    for (int c = threadIdx.x; c < width; c += blockDim.x) xr[c] += (sub(c) - mean) * rstd * post.w[c] + (post.b ? post.b[c] : 0.0f);     // a thread re-reads only what it wrote
     if (!next.w) return;
     mean = 0.0f; s = 0.0f;
     if (cn) {
@@ -278,7 +281,7 @@ __global__ void __launch_bounds__(256, SW_KEEP == 4 ? 4 : SW_KEEP == 2 ? 6 : 8) 
     for (int c = threadIdx.x; c < width; c += blockDim.x) { const float d = xr[c] - mean; s += d * d; }
     rstd = 1.0f / sqrtf(block_sum(s, red) / (float)width + next.eps);
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
-        const OT h = cvt<OT>((xr[c] - mean) * rstd * next.w[c] + (cn ? next.b[c] : 0.0f));
+        const OT h = cvt<OT>((xr[c] - mean) * rstd * next.w[c] + (next.b ? next.b[c] : 0.0f));
         op[(size_t)r * ld_op + c] = h;
         if (rn.w) srt[c] = ldf<OT>(&h);
     }
@@ -352,6 +355,108 @@ __global__ void __launch_bounds__(256) k_ret_post_all(RetBranch b, const float* 
         if (b.gated) { const float g = P[(size_t)r * ldp + b.g_off + c]; v *= b.gated == 2 ? sigmoidf_(g) : g * sigmoidf_(g); }
         out[(size_t)r * ld_out + b.a_off + c] = cvt<OT>(v);
     }
+}
+
+// ------------------------------------------------------------------------------------------------ convolution behind the projections
+struct ConvArgs {
+    int nq, nk, nv;              // channels: queries, keys (both convolved), values (appended as they are; 0: the values are the keys)
+    int off;                     // column of the first query channel in P; keys and values follow
+    int taps;
+    const float* w;              // [nq + nk][taps]
+    int max_ctx, k_ld, v_ld;     // cache rows
+};
+// y_t = sum_j w[c][j] u_(t - taps + 1 + j) of every query and key channel of P; queries -> Q [R][nq] (fp32), keys -> the slot's key cache.
+// Rows before the segment come from the slot's history `tail` [n_slots][taps - 1][nq + nk] (zeros after a reset = zeros before the
+// sequence).  A thread owns V neighbouring channels of `rows_per` consecutive rows and slides its window of `taps` values along them (TAPS 0:
+// any number of taps, read back from memory instead).  P keeps the projected values: other rows' windows and the history update read them.
+// every_one: each segment is one row, so the thread that has read a channel's history also writes its update.
+template <int V> __device__ __forceinline__ void cv_load(const float* __restrict__ p, float (&v)[V]) {
+    if (V == 4) { const float4 t = *reinterpret_cast<const float4*>(p); v[0] = t.x; v[V > 1 ? 1 : 0] = t.y; v[V > 2 ? 2 : 0] = t.z; v[V > 3 ? 3 : 0] = t.w; }
+    else v[0] = *p;
+}
+template <typename T> __device__ __forceinline__ void cv_store(T* p, const float (&v)[4]) { store4(p, v[0], v[1], v[2], v[3]); }
+template <typename T> __device__ __forceinline__ void cv_store(T* p, const float (&v)[1]) { *p = cvt<T>(v[0]); }
+template <typename OT, int V, int TAPS>
+__global__ void __launch_bounds__(128) k_qk_conv(PassTables t, ConvArgs b, const float* __restrict__ P, int ldp, int R, int rows_per, float* __restrict__ tail,
+                                                 float* __restrict__ Q, OT* __restrict__ kc, OT* __restrict__ vc, int every_one) {
+    const int nc = b.nq + b.nk, c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+    if (c >= nc + b.nv) return;
+    const int r0 = blockIdx.x * rows_per, r1 = min(R, r0 + rows_per);
+    const float* p = P + b.off + c;
+    if (c >= nc) {
+        for (int r = r0; r < r1; r++) {
+            float u[V];
+            cv_load<V>(p + (size_t)r * ldp, u);
+            cv_store(vc + ((size_t)t.seg_slot[t.row_seg[r]] * b.max_ctx + t.row_pos[r]) * b.v_ld + (c - nc), u);
+        }
+        return;
+    }
+    constexpr int NT = TAPS > 0 ? TAPS : 1;
+    float w[NT][V], u[NT][V];
+    if (TAPS > 0) {
+#pragma unroll
+        for (int j = 0; j < NT; j++)
+#pragma unroll
+            for (int i = 0; i < V; i++) w[j][i] = b.w[(size_t)(c + i) * NT + j];
+    }
+    int seg = -1, row0 = 0, slot = 0;
+    for (int r = r0; r < r1; r++) {
+        float y[V];
+        const bool fresh = t.row_seg[r] != seg;
+        if (fresh) { seg = t.row_seg[r]; row0 = t.seg_row0[seg]; slot = t.seg_slot[seg]; }
+        float* tl = tail + (size_t)slot * (b.taps - 1) * nc + c;
+        if (TAPS > 0) {
+            if (fresh) {
+#pragma unroll
+                for (int j = 0; j < NT - 1; j++) {
+                    const int src = r - (NT - 1) + j;
+                    if (src >= row0) cv_load<V>(p + (size_t)src * ldp, u[j]);
+                    else {
+#pragma unroll
+                        for (int i = 0; i < V; i++) u[j][i] = tl[(size_t)(src - row0 + NT - 1) * nc + i];
+                    }
+                }
+            }
+            cv_load<V>(p + (size_t)r * ldp, u[NT - 1]);
+#pragma unroll
+            for (int i = 0; i < V; i++) y[i] = 0.0f;
+#pragma unroll
+            for (int j = 0; j < NT; j++)
+#pragma unroll
+                for (int i = 0; i < V; i++) y[i] = fmaf(w[j][i], u[j][i], y[i]);
+#pragma unroll
+            for (int j = 0; j < NT - 1; j++)
+#pragma unroll
+                for (int i = 0; i < V; i++) u[j][i] = u[j + 1][i];
+            if (every_one && !t.slots[slot].stopped) {
+#pragma unroll
+                for (int j = 0; j < NT - 1; j++)
+#pragma unroll
+                    for (int i = 0; i < V; i++) tl[(size_t)j * nc + i] = u[j][i];
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < V; i++) y[i] = 0.0f;
+            for (int j = 0; j < b.taps; j++) {
+                const int src = r - (b.taps - 1) + j;
+#pragma unroll
+                for (int i = 0; i < V; i++)
+                    y[i] = fmaf(b.w[(size_t)(c + i) * b.taps + j], src >= row0 ? p[(size_t)src * ldp + i] : tl[(size_t)(src - row0 + b.taps - 1) * nc + i], y[i]);
+            }
+        }
+        if (c < b.nq) cv_store(Q + (size_t)r * b.nq + c, y);
+        else cv_store(kc + ((size_t)slot * b.max_ctx + t.row_pos[r]) * b.k_ld + (c - b.nq), y);
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ ungated feed-forward
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
+// act = gelu(G) -> operand [R][ld_out], zero-padded (grid: rows x column groups; few rows spread their columns over many CTAs)
+template <typename OT>
+__global__ void k_gelu_rows(const float* __restrict__ G, int ff, OT* __restrict__ out, int ld_out) {
+    const int r = blockIdx.x;
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < ld_out; c += gridDim.y * blockDim.x)
+        out[(size_t)r * ld_out + c] = cvt<OT>(c < ff ? gelu_erf(G[(size_t)r * ff + c]) : 0.0f);
 }
 
 }  // namespace seq

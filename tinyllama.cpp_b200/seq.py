@@ -14,9 +14,10 @@ LIB_PATH = HERE / "libgten_b200_seq.so"
 BF16, F32 = 0, 1
 MIX_SIGMOID_ATTN, MIX_RETENTION, MIX_MINGRU, MIX_SOFTMAX_ATTN, MIX_LATENT_ATTN = 1, 2, 3, 4, 5
 BLOCK_PARALLEL, BLOCK_POSTNORM, BLOCK_PRENORM, BLOCK_SANDWICH = 0, 1, 2, 3
-FF_GEGLU, FF_POLYNORM, FF_EXPERTS, FF_GATED_EXPERTS, FF_SWIGLU, FF_GROUP_EXPERTS = 0, 1, 2, 3, 4, 5
-NORM_RMS, NORM_DYT, NORM_LAYER = 0, 1, 2
+FF_GEGLU, FF_POLYNORM, FF_EXPERTS, FF_GATED_EXPERTS, FF_SWIGLU, FF_GROUP_EXPERTS, FF_GELU = 0, 1, 2, 3, 4, 5, 6
+NORM_RMS, NORM_DYT, NORM_LAYER, NORM_LAYER_NB = 0, 1, 2, 3
 ROT_HALVES, ROT_INTERLEAVED = 0, 1
+ROT_SCALE_WAVES, ROT_SCALE_YARN = 0, 1
 MODE_BY_NAME = {"bfloat16": BF16, "bf16": BF16, "float32": F32, "fp32": F32}
 
 
@@ -31,7 +32,8 @@ class BranchC(C.Structure):
                 ("rot_factor", C.c_float), ("rot_low", C.c_float), ("rot_high", C.c_float), ("rot_original", C.c_float), ("softcap", C.c_float),
                 ("window", C.c_int), ("pool", C.c_int), ("sink", C.c_int), ("kv_from", C.c_int),
                 ("rope_dim", C.c_int), ("kv_rank", C.c_int), ("q_rank", C.c_int),
-                ("chunk", C.c_int), ("maps", C.c_int), ("diff", C.c_float), ("bias", C.c_int), ("act", C.c_int), ("rot_divide", C.c_float)]
+                ("chunk", C.c_int), ("maps", C.c_int), ("diff", C.c_float), ("bias", C.c_int), ("act", C.c_int), ("rot_divide", C.c_float),
+                ("rot_scaling", C.c_int), ("conv", C.c_int), ("v_from_k", C.c_int), ("keep_first", C.c_int), ("slopes", C.c_int), ("out_bias", C.c_int)]
 
 
 class LayerC(C.Structure):
@@ -44,7 +46,7 @@ class ConfigC(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("vocab", "width", "n_layers")] + [("eps", C.c_float)] + \
                [(n, C.c_int) for n in ("taps", "bigram_buckets", "bigram_mul_prev", "bigram_mul_cur", "loop_start", "loop_stop", "loop_times",
                                        "mode", "n_slots", "max_ctx", "max_rows")] + [("embed_scale", C.c_float), ("final_norm", C.c_int), ("streams", C.c_int),
-                                                                                     ("logit_softcap", C.c_float)]
+                                                                                     ("logit_softcap", C.c_float), ("logit_scale", C.c_float), ("tied_head", C.c_int)]
 
 
 SYMBOLS = ["gtb_seq_create", "gtb_seq_destroy", "gtb_seq_set_tensor", "gtb_seq_finalize", "gtb_seq_n_runs", "gtb_seq_slot_reset",
@@ -128,7 +130,7 @@ class SeqModel:
 
     def __init__(self, desc: dict, mode: int, n_slots: int, max_ctx: int, max_rows: int = 0):
         """desc: the flat description a model family's config reader produces (see reninex.describe, robopel.describe, nanotar.describe,
-        vulosun.describe)."""
+        vulosun.describe, bisodra.describe)."""
         self.desc, self.mode, self.n_slots, self.max_ctx = desc, mode, n_slots, max_ctx
         self.vocab, self.width = desc["vocab"], desc["width"]
         layers = (LayerC * len(desc["layers"]))()
@@ -153,6 +155,8 @@ class SeqModel:
                 bc.rope_dim, bc.kv_rank, bc.q_rank = b.get("rope_dim", 0), b.get("kv_rank", 0), b.get("q_rank", 0)
                 bc.chunk, bc.maps, bc.diff = b.get("chunk", 0), b.get("maps", 1), b.get("diff", 0.0)
                 bc.bias, bc.act, bc.rot_divide = int(b.get("bias", 0)), int(b.get("act", 0)), b.get("rot_divide", 0.0)
+                bc.rot_scaling, bc.conv, bc.v_from_k = b.get("rot_scaling", ROT_SCALE_WAVES), b.get("conv", 0), int(b.get("v_from_k", 0))
+                bc.keep_first, bc.slopes, bc.out_bias = b.get("keep_first", 0), int(b.get("slopes", 0)), int(b.get("out_bias", 0))
                 if b.get("decay") is not None:
                     arr = (C.c_float * len(b["decay"]))(*b["decay"])
                     self._keep.append(arr)
@@ -161,7 +165,8 @@ class SeqModel:
         cfg = ConfigC(desc["vocab"], desc["width"], len(desc["layers"]), desc["eps"], desc.get("taps", 0),
                       bg["buckets"] if bg else 0, bg["mul_prev"] if bg else 0, bg["mul_cur"] if bg else 0,
                       lp["start"] if lp else 0, lp["stop"] if lp else 0, lp["times"] if lp else 0, mode, n_slots, max_ctx, max_rows,
-                      desc.get("embed_scale", 1.0), int(desc.get("final_norm", 0)), int(desc.get("streams", 0)), float(desc.get("logit_softcap", 0.0)))
+                      desc.get("embed_scale", 1.0), int(desc.get("final_norm", 0)), int(desc.get("streams", 0)), float(desc.get("logit_softcap", 0.0)),
+                      float(desc.get("logit_scale", 1.0)), int(desc.get("tied_head", 0)))
         self.h = C.c_void_p()
         check(lib().gtb_seq_create(C.byref(self.h), C.byref(cfg), layers))
         n = C.c_int()
