@@ -361,7 +361,7 @@ __global__ void __launch_bounds__(128) k_sattn_prep(PassTables t, SoftAttn b, fl
     const int slot = t.seg_slot[t.row_seg[r]], pos = t.row_pos[r];
     float* p = P + (size_t)r * ldp;
     const size_t crow = (size_t)slot * b.max_ctx + pos;
-    const int M = sa_maps(b), nq = b.heads * M, nk = b.own_kv ? b.kv_heads * M : 0, nkv = b.own_kv ? b.kv_heads : 0, half = b.rot_dims / 2;
+    const int M = sa_maps(b), nq = b.heads * M, nk = b.own_kv ? b.kv_heads * M : 0, nkv = b.own_kv && !b.v_is_k ? b.kv_heads : 0, half = b.rot_dims / 2;
     const float fpos = (float)pos;
     for (int u = blockIdx.y * nw + wid; u < nq + nk + nkv; u += gridDim.y * nw) {
         if (u < nq + nk) {
