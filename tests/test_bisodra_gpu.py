@@ -578,7 +578,7 @@ def oracle_greedy(cfg, W, prompt, n_new):
 
 def test_greedy_generation_through_the_scheduler(lib):
     from tinyllama_cpp_b200.scheduler import generate
-    cfg = BI.make_config(vocab=64, width=64)
+    cfg = BI.make_config(vocab=64, width=64, logit_scale=-0.5)      # (a tied head with a positive scale mostly repeats its last token)
     m, W = make(lib, cfg, "float32", seed=41, n_slots=2, gain=2.0)
     prompts = [toks(80 + i, n, 64) for i, n in enumerate((19, 3, 40))]     # three requests, two slots: one waits
     outs = generate(m, prompts, 12, chunk=8, burst=5)
@@ -587,11 +587,12 @@ def test_greedy_generation_through_the_scheduler(lib):
         assert len(o) == 12
         k = int(np.argmax(o != want)) if np.any(o != want) else 12
         assert k == 12 or margin[k] < 1e-3, (o, want, margin)
+        assert len(set(o.tolist())) > 2
 
 
 def test_device_decode_loop_equals_host_fed_steps(lib):
-    """The graph-replayed loop, across a window's edge, and a sequence that stops while another goes on: the stopped slot's state stays."""
-    cfg = BI.make_config(vocab=64, width=64)
+    """The graph-replayed loop, across a window's edge."""
+    cfg = BI.make_config(vocab=64, width=64, logit_scale=-0.5)
     m, _ = make(lib, cfg, "float32", seed=43, n_slots=3, gain=2.0)
     p0, p1 = toks(90, 11, 64), toks(91, 30, 64)
     nxt = m.step_greedy([(0, p0), (1, p1)])
@@ -606,7 +607,26 @@ def test_device_decode_loop_equals_host_fed_steps(lib):
         cur = int(m.step_greedy([(2, [cur])])[0])
         host.append(cur)
     assert host == dev[1].tolist()
-    assert m.position(1) == 30 + 20
+    assert m.position(1) == 30 + 20 and len(set(host)) > 2
+
+
+def test_a_sequence_that_stops_beside_one_that_goes_on(lib):
+    """Sequence 0 samples the end id in the device loop: it repeats that id and its position stays, sequence 1 is not disturbed, and the slot
+    starts afresh after a reset (its cache and convolution history were written until it stopped)."""
+    cfg = BI.make_config(vocab=64, width=64, logit_scale=-0.5)
+    m, W = make(lib, cfg, "float32", seed=44, n_slots=2, gain=2.0)
+    p0, p1 = toks(92, 11, 64), toks(93, 30, 64)
+    nxt = m.step_greedy([(0, p0), (1, p1)])
+    free = m.decode([0, 1], 12)
+    eos = next(int(e) for e in free[0] if e not in free[1] and e != nxt[0] and e != nxt[1])
+    first = free[0].tolist().index(eos)
+    m.reset(0), m.reset(1)
+    m.step_greedy([(0, p0), (1, p1)])
+    got = m.decode([0, 1], 12, eos)
+    assert (got[0][first:] == eos).all() and got[0][:first].tolist() == free[0][:first].tolist() and np.array_equal(got[1], free[1])
+    assert m.position(0) == 11 + 1 + first and m.position(1) == 30 + 12
+    m.reset(0)
+    assert rel(m.step([(0, p1[:9])], range(9)), R.forward(cfg, W, p1[:9])) < TOL["float32"]
 
 
 def test_missing_and_misshapen_tensors_are_named(lib):
@@ -633,7 +653,7 @@ def test_command_line_generation_and_trace_replay(lib, tmp_path):
     import sys
     from pathlib import Path
     root = Path(__file__).resolve().parent.parent
-    cfg = BI.make_config(vocab=64, width=64)
+    cfg = BI.make_config(vocab=64, width=64, logit_scale=-0.5)
     t = BI.synth_tensors(BI.describe(cfg), 71, gain=2.0)
     BI.write_checkpoint(tmp_path / "m", cfg, t)
     W = {k: R.to_float(v) for k, v in t.items()}

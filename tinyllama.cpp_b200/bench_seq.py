@@ -4,7 +4,8 @@ family, beside Reninex (the closest existing model: same library, same width and
 family beside Robopel (the closest existing model: softmax attention with a window, a sink and an output gate, routed experts) at the same
 widths and layer count.  `bench.py --workload vulosun`: the Vulosun family beside Robopel (the closest existing model: sequential sublayers
 with norms on their outputs, softmax attention with a sink, a gate and a shared cache, squared-ReLU experts) at the same widths and layer
-count.  Timed with CUDA events on each library's own stream,
+count.  `bench.py --workload bisodra`: the Bisodra family beside Vulosun (the same layer style) and Nanotar (the same latent attention) at the
+same widths and layer count.  Timed with CUDA events on each library's own stream,
 after warm-up; the weights of one pass (hundreds of MB) are larger than L2, so every pass streams them from HBM."""
 from __future__ import annotations
 
@@ -488,6 +489,137 @@ def run_vulosun(args, root, clock_sampler) -> None:
                       "steps": iters, "warmup": warm, "ms_per_step": head["prefill"]["ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
                       "dtype": "bf16 operands, fp32 accumulation; fp32 stream, norms, scores, recurrent state, router", "data": "synthetic",
                       "config": {"workload": f"Vulosun {head['size']} x {head['layers']} layers, random weights: prefill of {T} tokens; decode at that context",
+                                 "l2": "weights of a pass exceed L2"},
+                      "detail": res, "gpu_launches": head["prefill_launches"], "clocks": clk.summary()}), flush=True)
+
+
+BISODRA_SIZES = {
+    # width, dense ff (two matrices); windowed heads / kv x dim, taps, window, kept tokens; latent heads x (plain + rotated | value), ranks
+    "w2048": dict(width=2048, ff=8192, heads=32, kv=8, dim=64, conv=4, window=1024, keep=64, l_heads=16, l_dim=96, l_rot=32, l_vdim=128, kv_rank=512, q_rank=768),
+    "w1024": dict(width=1024, ff=4096, heads=16, kv=4, dim=64, conv=4, window=512, keep=64, l_heads=8, l_dim=96, l_rot=32, l_vdim=128, kv_rank=256, q_rank=384),
+}
+
+
+def bisodra_config(name, vocab=32000):
+    """Four layers: windowed attention, latent attention, windowed attention, latent attention on layer 1's latents; all with a dense feed-forward."""
+    from . import bisodra as BI
+    z = BISODRA_SIZES[name]
+    win = dict(heads=z["heads"], kv_heads=z["kv"], dim=z["dim"], conv=z["conv"], window=z["window"], keep_first=z["keep"])
+    lat = dict(heads=z["l_heads"], dim=z["l_dim"], rot_dim=z["l_rot"], vdim=z["l_vdim"], kv_rank=z["kv_rank"], q_rank=z["q_rank"], rot_base=500000.0, yarn=(4.0, 1024.0, 32.0, 1.0))
+    ml = lambda: BI.dense_mlp(z["ff"])
+    layers = [BI.windowed_layer(mlp=ml(), **win), BI.latent_layer(mlp=ml(), **lat), BI.windowed_layer(mlp=ml(), **win), BI.latent_layer(kv_from=1, mlp=ml(), **lat)]
+    return BI.make_config(vocab=vocab, width=z["width"], layers=layers, eps=1e-6, embed_scale=16.0, logit_scale=0.25)
+
+
+def bisodra_counts(desc, T):
+    """(weights every token multiplies, FLOPs of the attention's own arithmetic for a T-token prompt, bytes of weights a decode step of one
+    sequence reads); attention counts the keys a row really sees."""
+    from .seq import MIX_LATENT_ATTN
+    W, params, mix = desc["width"], 0, 0.0
+    for l in desc["layers"]:
+        b = l["branches"][0]
+        H, V = b["heads"], b["vdim"]
+        if b["kind"] == MIX_LATENT_ATTN:
+            hd = b["dim"] + b["rope_dim"]
+            params += W * (b["q_rank"] + (b["kv_rank"] + b["rope_dim"] if b["kv_from"] < 0 else 0) + 2 * H * V) + b["q_rank"] * H * hd + b["kv_rank"] * H * (b["dim"] + V)
+            mix += 2.0 * H * (hd + V) * T * (T + 1) / 2
+        else:
+            params += W * ((H + b["kv_heads"]) * b["dim"] + 2 * H * V)
+            n, keep = b.get("window", 0) or T, b.get("keep_first", 0)
+            mix += 2.0 * H * (b["dim"] + V) * sum(min(i + 1, n) + min(keep, max(0, i + 1 - n)) for i in range(T))
+        params += 2 * W * l["ff"]
+    return params + desc["vocab"] * W, mix, 2 * (params + desc["vocab"] * W)
+
+
+def bisodra_section(torch, name, T, iters, warmup, peaks):
+    from . import bisodra as BI, seq
+    desc = BI.describe(bisodra_config(name))
+    t0 = time.time()
+    rng = np.random.default_rng(0)
+    tensors = {}
+    for k, shape in BI.tensor_shapes(desc).items():              # cheap random bf16 patterns of the right scale
+        n = int(np.prod(shape))
+        leaf = k.split(".")[-1]
+        if leaf == "b":
+            a = np.zeros(n, np.uint16)
+        elif leaf.startswith("norm"):
+            a = np.full(n, 0x3F80, np.uint16)
+        else:
+            std = 1.0 / 16.0 if k == "embed" else (0.5 if leaf == "conv" else 1.0 / np.sqrt(shape[-1]))
+            a = BI.st.f32_to_bf16_bits(rng.standard_normal(n, np.float32) * np.float32(std))
+        tensors[k] = a.reshape(shape)
+    n_slots = 8
+    m = seq.SeqModel(desc, seq.BF16, n_slots, T + 64, max_rows=T).load(tensors)
+    stream = torch.cuda.ExternalStream(seq.stream_handle(), device=torch.device("cuda", 0))
+    prompt = rng.integers(0, desc["vocab"], T).astype(np.int32)
+    params, mix, dec_bytes = bisodra_counts(desc, T)
+    out = {"size": name, "layers": len(desc["layers"]), "params_matmul_per_token": params, "weight_bytes": m.weight_bytes(), "setup_s": round(time.time() - t0, 1)}
+
+    def prefill():
+        m.reset(0)
+        m.step([(0, prompt)], [T - 1])
+    l0 = seq.launch_count()
+    prefill()
+    out["prefill_launches"] = seq.launch_count() - l0
+    ms = _events(torch, stream, prefill, iters, warmup)
+    flops = 2.0 * T * params - 2.0 * (T - 1) * desc["vocab"] * desc["width"] + mix
+    out["prefill"] = {"T": T, "ms": ms, "tokens_per_s": T / ms * 1e3, "tflops": flops / ms * 1e-9, "frac_of_bf16_peak": flops / ms * 1e-9 / peaks["tflops"],
+                      "note": "includes the host->device copy of the prompt and the device->host copy of the last row's logits"}
+
+    def chunked():                                                # the same prompt in four portions: every portion expands the latents before it again
+        m.reset(0)
+        for i in range(0, T, T // 4):
+            m.step([(0, prompt[i:i + T // 4])], [T // 4 - 1])
+    out["prefill_in_4_portions_ms"] = _events(torch, stream, chunked, max(3, iters // 2), 2)
+    for s in range(n_slots):
+        m.reset(s)
+        m.step_greedy([(s, prompt[: T - 40])])
+    state_bytes = m.state_bytes_per_slot() * (T - 40) / (T + 64)
+    for nseq in (1, 8):
+        slots, steps = list(range(nseq)), 8
+        m.decode(slots, 2)
+        t_ms = []
+        with torch.cuda.stream(stream):
+            for _ in range(3):
+                a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                a.record(stream)
+                m.decode(slots, steps)
+                b.record(stream)
+                torch.cuda.synchronize()
+                t_ms.append(a.elapsed_time(b) / steps)
+        ms = float(np.median(t_ms))
+        out[f"decode_{nseq}"] = {"ms_per_step": ms, "tokens_per_s": nseq / ms * 1e3, "bytes_per_step_one_sequence": dec_bytes, "gbs": dec_bytes / ms * 1e-6,
+                                 "frac_of_hbm_peak": dec_bytes / ms * 1e-6 / peaks["hbm_gbs"],
+                                 "note": "bytes: the weights a step reads; sequences add their cached keys and latents"}
+    out["state_bytes_per_slot_at_T"] = state_bytes
+    m.close()
+    return out
+
+
+def run_bisodra(args, root, clock_sampler) -> None:
+    """`--workload bisodra`: Bisodra at two sizes, Vulosun and Nanotar at the same widths and layer count in the same call."""
+    import torch
+    from . import build, seq
+    build.build(target="seq")
+    torch.cuda.set_device(0)
+    peaks = _peaks(root)
+    seq.init(0)
+    T = 2048
+    iters = max(3, min(args.steps if args.steps != 512 else 5, 20))
+    warm = max(args.warmup if args.warmup != 16 else 3, 3)
+    res = {"bisodra": [], "vulosun_same_width": [], "nanotar_same_width": [], "peaks": peaks}
+    with clock_sampler(0) as clk:
+        for name in BISODRA_SIZES:
+            res["bisodra"].append(bisodra_section(torch, name, T, iters, warm, peaks))
+        for name in VULOSUN_SIZES:
+            res["vulosun_same_width"].append(vulosun_section(torch, name, T, iters, warm, peaks))
+        for name in NANOTAR_SIZES:
+            res["nanotar_same_width"].append(nanotar_section(torch, name, T, iters, warm, peaks))
+    head = res["bisodra"][0]
+    print(json.dumps({"metric": "bisodra_prefill_tokens_per_s", "value": head["prefill"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+                      "steps": iters, "warmup": warm, "ms_per_step": head["prefill"]["ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+                      "dtype": "bf16 operands, fp32 accumulation; fp32 stream, norms, convolution, scores", "data": "synthetic",
+                      "config": {"workload": f"Bisodra {head['size']} x {head['layers']} layers, random weights: prefill of {T} tokens; decode at that context",
                                  "l2": "weights of a pass exceed L2"},
                       "detail": res, "gpu_launches": head["prefill_launches"], "clocks": clk.summary()}), flush=True)
 

@@ -837,6 +837,16 @@ int run_sandwich_layer(gtb_seq_model* m, const PassTables& t, int R, int S, cons
             if (rc > 0) return rc;
             if (rc == 0) { ctx().launches++; act_done = true; }
         }
+        if (!act_done && R <= 8) {          // few rows: the activation leaves the weight-streaming product
+            const OT* a = opA;
+            const dim3 grid((l.ff + 3) / 4);
+            if (R <= 1) k_gemv_rows<OT, 1, 4, true, OT><<<grid, 256, 0, st>>>(a, wp, l.w_up, wp, opC, l.kfp, R, l.ff, wp, nullptr, 0);
+            else if (R <= 2) k_gemv_rows<OT, 2, 4, true, OT><<<grid, 256, 0, st>>>(a, wp, l.w_up, wp, opC, l.kfp, R, l.ff, wp, nullptr, 0);
+            else if (R <= 4) k_gemv_rows<OT, 4, 4, true, OT><<<grid, 256, 0, st>>>(a, wp, l.w_up, wp, opC, l.kfp, R, l.ff, wp, nullptr, 0);
+            else k_gemv_rows<OT, 8, 4, true, OT><<<grid, 256, 0, st>>>(a, wp, l.w_up, wp, opC, l.kfp, R, l.ff, wp, nullptr, 0);
+            GTB_LAUNCHED();
+            act_done = true;
+        }
         if (!act_done) {
             rc = product<OT>(m, opA, wp, l.w_up, wp, m->G, l.ff, R, l.ff, wp, nullptr, 0);
             if (rc) return rc;

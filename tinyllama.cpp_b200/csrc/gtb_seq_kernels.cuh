@@ -101,6 +101,7 @@ __device__ __forceinline__ float gelu_tanh(float z) {
     const float c = 0.7978845608028654f;      // sqrt(2/pi)
     return 0.5f * z * (1.0f + tanhf(c * (z + 0.044715f * z * z * z)));
 }
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
 
 // ------------------------------------------------------------------------------------------------ plan / commit
 // row tables of a pass from the slots' device-side state.  from_pending: rows take their token from the slot (decode loop).
@@ -302,8 +303,10 @@ template <> __device__ __forceinline__ void load8<bf16>(const bf16* p, float (&v
 #pragma unroll
     for (int i = 0; i < 4; i++) { v[2 * i] = __uint_as_float(w[i] << 16); v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
 }
-template <typename AT, int MR, int NC>
-__global__ void __launch_bounds__(256) k_gemv_rows(const AT* __restrict__ A, int lda, const bf16* __restrict__ W, int ldw, float* __restrict__ C, int ldc,
+// OUT float: C (fp32) as above.  GELU: gelu(A . W^T), erf form, as the next product's operand (OUT = AT) -- the activation of an ungated
+// feed-forward; no bias, no accumulation.
+template <typename AT, int MR, int NC, bool GELU = false, typename OUT = float>
+__global__ void __launch_bounds__(256) k_gemv_rows(const AT* __restrict__ A, int lda, const bf16* __restrict__ W, int ldw, OUT* __restrict__ C, int ldc,
                                                    int M, int N, int K, const float* __restrict__ bias, int accumulate) {
     __shared__ float red[8][MR * NC];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -350,9 +353,13 @@ __global__ void __launch_bounds__(256) k_gemv_rows(const AT* __restrict__ A, int
             float o = 0.0f;
 #pragma unroll
             for (int w = 0; w < 8; w++) o += red[w][threadIdx.x];
-            if (bias) o += bias[n0 + c];
-            if (accumulate) o += C[(size_t)m * ldc + n0 + c];
-            C[(size_t)m * ldc + n0 + c] = o;
+            if constexpr (GELU) {
+                C[(size_t)m * ldc + n0 + c] = cvt<OUT>(gelu_erf(o));
+            } else {
+                if (bias) o += bias[n0 + c];
+                if (accumulate) o += C[(size_t)m * ldc + n0 + c];
+                C[(size_t)m * ldc + n0 + c] = o;
+            }
         }
     }
 }

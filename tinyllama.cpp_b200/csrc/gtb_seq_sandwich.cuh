@@ -450,7 +450,6 @@ __global__ void __launch_bounds__(128) k_qk_conv(PassTables t, ConvArgs b, const
 }
 
 // ------------------------------------------------------------------------------------------------ ungated feed-forward
-__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
 // act = gelu(G) -> operand [R][ld_out], zero-padded (grid: rows x column groups; few rows spread their columns over many CTAs)
 template <typename OT>
 __global__ void k_gelu_rows(const float* __restrict__ G, int ff, OT* __restrict__ out, int ld_out) {
