@@ -508,7 +508,7 @@ def bisodra_config(name, vocab=32000):
     lat = dict(heads=z["l_heads"], dim=z["l_dim"], rot_dim=z["l_rot"], vdim=z["l_vdim"], kv_rank=z["kv_rank"], q_rank=z["q_rank"], rot_base=500000.0, yarn=(4.0, 1024.0, 32.0, 1.0))
     ml = lambda: BI.dense_mlp(z["ff"])
     layers = [BI.windowed_layer(mlp=ml(), **win), BI.latent_layer(mlp=ml(), **lat), BI.windowed_layer(mlp=ml(), **win), BI.latent_layer(kv_from=1, mlp=ml(), **lat)]
-    return BI.make_config(vocab=vocab, width=z["width"], layers=layers, eps=1e-6, embed_scale=16.0, logit_scale=0.25)
+    return BI.make_config(vocab=vocab, width=z["width"], layers=layers, eps=1e-6, embed_scale=8.0, logit_scale=0.5)
 
 
 def bisodra_counts(desc, T):
@@ -545,7 +545,7 @@ def bisodra_section(torch, name, T, iters, warmup, peaks):
         elif leaf.startswith("norm"):
             a = np.full(n, 0x3F80, np.uint16)
         else:
-            std = 1.0 / 16.0 if k == "embed" else (0.5 if leaf == "conv" else 1.0 / np.sqrt(shape[-1]))
+            std = 0.125 if k == "embed" else (0.5 if leaf == "conv" else 1.0 / np.sqrt(shape[-1]))
             a = BI.st.f32_to_bf16_bits(rng.standard_normal(n, np.float32) * np.float32(std))
         tensors[k] = a.reshape(shape)
     n_slots = 8

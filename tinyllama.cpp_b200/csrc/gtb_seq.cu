@@ -17,7 +17,9 @@
 //    block of 2 ff rows ([experts][2 ff][width]), the shared expert's gate as one more row of the router matrix.
 //  * sandwich layers (GTB_BLOCK_SANDWICH) run like post-norm layers with a norm on both sides of each sublayer: one kernel per sublayer
 //    boundary adds norm_b(sublayer output) to the stream and writes the next sublayer's normalised input.  Their mixers are the branch
-//    kernels of the other styles (softmax attention, retention) side by side, each weighted by out_scale in the out-projection operand.
+//    kernels of the other styles (softmax attention, retention) side by side, each weighted by out_scale in the out-projection operand --
+//    or latent attention alone.  Queries and keys that pass a convolution behind their projections leave the raw projection in place (its
+//    last rows become the slot's history): the queries go to a buffer of their own, the keys to the cache.
 //    Group-limited experts reuse the stacked layout of the post-norm experts; the shared expert is cut along its inner width into parts of
 //    one expert's size that follow the routed experts in the same stacks, so every row simply has `top + parts` choices.
 #include <math.h>
