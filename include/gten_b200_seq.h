@@ -25,10 +25,12 @@ extern "C" {
 #endif
 
 enum { GTB_SEQ_BF16 = 0, GTB_SEQ_F32 = 1 };                       /* compute mode */
-enum { GTB_MIX_SIGMOID_ATTN = 1, GTB_MIX_RETENTION = 2, GTB_MIX_MINGRU = 3, GTB_MIX_SOFTMAX_ATTN = 4, GTB_MIX_LATENT_ATTN = 5 };   /* branch kinds of a token mixer */
+enum { GTB_MIX_SIGMOID_ATTN = 1, GTB_MIX_RETENTION = 2, GTB_MIX_MINGRU = 3, GTB_MIX_SOFTMAX_ATTN = 4, GTB_MIX_LATENT_ATTN = 5, GTB_MIX_MLSTM = 6, GTB_MIX_DELTA = 7,
+       GTB_MIX_SSM = 8 };   /* branch kinds of a token mixer */
 enum { GTB_BLOCK_PARALLEL = 0, GTB_BLOCK_POSTNORM = 1, GTB_BLOCK_PRENORM = 2, GTB_BLOCK_SANDWICH = 3 };   /* layer styles */
 enum { GTB_FF_GEGLU = 0, GTB_FF_POLYNORM = 1, GTB_FF_EXPERTS = 2, GTB_FF_GATED_EXPERTS = 3, GTB_FF_SWIGLU = 4, GTB_FF_GROUP_EXPERTS = 5, GTB_FF_GELU = 6 };   /* feed-forward kinds */
 enum { GTB_NORM_RMS = 0, GTB_NORM_DYT = 1, GTB_NORM_LAYER = 2, GTB_NORM_LAYER_NB = 3 };   /* norm of a pre-norm / sandwich layer and of the model's output (NB: no bias) */
+enum { GTB_ROUTE_LOGISTIC = 0, GTB_ROUTE_SOFTMAX = 1 };           /* weights of GTB_FF_GATED_EXPERTS */
 enum { GTB_ROT_HALVES = 0, GTB_ROT_INTERLEAVED = 1 };             /* which entries a rotary pair takes: (i, i + dims/2) or (2i, 2i + 1) */
 enum { GTB_ROT_SCALE_WAVES = 0, GTB_ROT_SCALE_YARN = 1 };         /* how rot_factor > 0 rescales the frequencies (see rot_scaling) */
 
@@ -81,6 +83,19 @@ enum { GTB_ROT_SCALE_WAVES = 0, GTB_ROT_SCALE_YARN = 1 };         /* how rot_fac
  *    maps 2).  keep_first > 0: tokens j < keep_first stay visible outside the window or chunk, at their true distance (not with pool).  slopes: 2^(-8 (h + 1) / heads) (i - j) is taken off head h's scores (not with pool).
  *    sink 2: the sink's score is 0 for every head (no tensor): the denominator holds one more 1.  out_bias: the out projection adds the
  *    vector o.b (single-branch layers, both attention kinds).
+ *  Recurrent mixers of sandwich layers (fp32 state per slot, gates, decays, step sizes and unit norms in fp32):
+ *  GTB_MIX_MLSTM: per head log gates i = gate_cap tanh((i h + i.b) / gate_cap), f = log logistic(gate_cap tanh((f h + f.b) / gate_cap)); with
+ *    m_0 = 0, m_t = max(f + m_(t-1), i): S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k v^T, the vector n_t likewise with k alone, both from
+ *    zero; o = S_t^T q / (max(|n_t . q|, exp(-m_t)) + 1e-6), q scaled by `scale`; per head o to unit RMS (eps of the model), times `norm`
+ *    [heads * vdim], times logistic(g h).  Tensors q, k, v, g, i, i.b, f, f.b, norm, o.
+ *  GTB_MIX_DELTA: q, k (kv_heads heads; head h uses h / (heads / kv_heads)) and v each pass a causal convolution of `conv` taps per channel (as
+ *    below, no bias) and silu; q and k divided by sqrt(sum of squares + 1e-6), q times `scale`; g_t = exp(-exp(A_log) softplus(a h + dt_bias)),
+ *    beta = logistic(b h) per head; S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q; per head o to unit RMS times `norm` [vdim], times
+ *    silu(g h).  Tensors q, k, v, q.conv, k.conv, v.conv, g, b, a, A_log, dt_bias, norm, o.
+ *  GTB_MIX_SSM: selective scan over `inner` channels with `state` numbers each: [x | z] = in h; x passes the convolution of `conv` taps with bias
+ *    conv.b and silu; [d | B | C] = x_proj x (dt_rank, state, state rows of tensor x), dt = softplus(dt d + dt.b), S[c][n] <- exp(-dt_c
+ *    exp(A_log[c][n])) S[c][n] + dt_c x_c B_n, y_c = sum_n S[c][n] C_n + D_c x_c; output o (y * silu(z)).  Tensors in, conv, conv.b, x, dt,
+ *    dt.b, A_log, D, o.
  *    retention -- act 1: q, k, v <- silu(q), silu(k), silu(v) before the recurrence; out_norm 2: the concatenated heads are scaled to
  *    unit RMS TOGETHER and multiplied by the weight `norm` [heads * vdim]; gated 2: times logistic(g h). */
 typedef struct {
@@ -113,6 +128,8 @@ typedef struct {
     int keep_first;                  /* first tokens of the sequence that stay visible whatever the window */
     int slopes;                      /* 1: head-wise slope times the distance is taken off the scores */
     int out_bias;                    /* 1: the out projection has a bias vector */
+    float gate_cap;                  /* GTB_MIX_MLSTM */
+    int inner, state, dt_rank;       /* GTB_MIX_SSM */
 } gtb_seq_branch;
 
 /* Tensors of layer i beyond its branches'.  Parallel blocks: "l<i>.norm1" (one gain), "l<i>.mlp.{gate,up,down}", "l<i>.canon{1,2}".
@@ -137,13 +154,14 @@ typedef struct {
                                       * (GTB_MIX_LATENT_ATTN);
                                       * GTB_BLOCK_SANDWICH: x += norm1b(mixer(norm1(x))); x += norm2b(ff(norm2(x))), four norms of kind norm_kind
                                       * (GTB_NORM_LAYER, GTB_NORM_LAYER_NB or GTB_NORM_RMS with a plain weight); one or two branches
-                                      * (GTB_MIX_SOFTMAX_ATTN, GTB_MIX_RETENTION), each weighted by its out_scale, or one GTB_MIX_LATENT_ATTN */
+                                      * (any kind but GTB_MIX_SIGMOID_ATTN, GTB_MIX_MINGRU), each weighted by its out_scale, or one GTB_MIX_LATENT_ATTN */
     int ff_kind;                     /* GTB_FF_GEGLU: down(gelu_tanh(gate h) * (up h)); GTB_FF_POLYNORM: down(a N(z) + b N(z^2) + c N(z^3) + e),
                                       * z = up h, N = unit RMS over the ff values, (a, b, c, e) = tensor mlp.act; GTB_FF_EXPERTS: router outputs
                                       * 0 .. experts-1 are experts e<i>.down(relu(e<i>.up h)^2), the `identity` outputs after them return h;
                                       * s = softmax(router h), the `top` largest s + correction are chosen and weighted with their s;
                                       * GTB_FF_GATED_EXPERTS: experts e<i>.down(silu(e<i>.gate h) * (e<i>.up h)); s = logistic(router h) in fp32, the
-                                      * `top` largest s are chosen (ties to the lower index) and weighted with s / (sum of the chosen s + 1e-20);
+                                      * `top` largest s are chosen (ties to the lower index) and weighted with s / (sum of the chosen s + 1e-20) (pre-norm and
+                                      * sandwich layers; see route_kind);
                                       * shared_ff > 0: an expert of that inner width runs for every row, times logistic(shared.sg h);
                                       * GTB_FF_SWIGLU: down(silu(gate h) * (up h));
                                       * GTB_FF_GROUP_EXPERTS: experts e<i>.down(relu(e<i>.up h)^2); s = logistic(router h) in fp32; the experts form
@@ -159,6 +177,12 @@ typedef struct {
     int shared_ff;
     int route_groups, route_keep;    /* GTB_FF_GROUP_EXPERTS (0 groups counts as 1, 0 kept as all) */
     float route_scale;
+    int route_kind;                  /* GTB_FF_GATED_EXPERTS: GTB_ROUTE_LOGISTIC, or GTB_ROUTE_SOFTMAX (largest router outputs chosen, weights = softmax
+                                      * over the chosen outputs) */
+    int join_norm;                   /* two-branch sandwich layers, 1: every branch has an out projection of its own, scaled to unit RMS over the width
+                                      * (eps of the model) times the weight "<branch>.out" [width]; the mixer's output is the mean of the two */
+    int weights_of;                  /* -1: tensors of its own; j: the layer IS layer j once more (the rest of the entry is not read) with a cache
+                                      * and state of its own; j must be an earlier layer with tensors of its own */
 } gtb_seq_layer;
 
 typedef struct {
@@ -172,7 +196,8 @@ typedef struct {
     int max_rows;                    /* rows per pass over the weights (longer steps are cut into passes); 0: default */
     float embed_scale;               /* embedding rows are multiplied by this (0 counts as 1) */
     int final_norm;                  /* 0: one gain; 1: weight vector stored around zero (1 + w); 2: Dynamic Tanh, tensors final.norm, final.norm.alpha, final.norm.b;
-                                      * 3: layer norm, tensors final.norm, final.norm.b; 4: layer norm without bias, tensor final.norm */
+                                      * 3: layer norm, tensors final.norm, final.norm.b; 4: layer norm without bias, tensor final.norm; 5: RMS norm, plain weight
+                                      * vector final.norm */
     int streams;                     /* pre-norm layers: copies of the residual stream under hyper-connections (all equal to the embedding output at
                                       * the start, summed at the end); 0: one stream, plain residual sum */
     float logit_softcap;             /* > 0: logits <- cap * tanh(logits / cap) */
@@ -215,7 +240,7 @@ int gtb_seq_last_logits(gtb_seq_t m, int seg, float* h_logits);
  * "tensor" (1, default: bf16 matrix products of >= "tensor_min_rows" rows on tcgen05; 0: SIMT kernels only),
  * "tensor_min_rows" (default 64), "graph" (1, default: gtb_seq_decode replays a CUDA graph per step),
  * "fused_attn" (1, default: tiled kernels of the mixers on prompt portions -- tensor-core attention in bf16 mode, chunked
- * retention and minGRU, expanded keys and values for latent attention; decode rows of latent attention on tensor cores in bf16 mode;
+ * retention and minGRU, chunked mLSTM and delta rule in bf16 mode, expanded keys and values for latent attention; decode rows of latent attention on tensor cores in bf16 mode;
  * 0: the row-at-a-time kernels), "grouped_experts" (1, default: rows sorted by expert and multiplied as groups
  * on passes of tensor_min_rows rows or more; 0: one weight stream per row and choice), "fused_norm" (1, default: norm and input convolution in one kernel on passes of 32 rows or more; 0: two kernels) */
 int gtb_seq_set_option(gtb_seq_t m, const char* name, int value);

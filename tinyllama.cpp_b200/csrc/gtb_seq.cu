@@ -38,6 +38,7 @@
 #include "gtb_seq_mixers_tiled.cuh"
 #include "gtb_seq_latent.cuh"
 #include "gtb_seq_sandwich.cuh"
+#include "gtb_seq_recur.cuh"
 
 using namespace gtb;
 using namespace gtb::seq;
@@ -80,6 +81,13 @@ struct BranchW {
     float* d_slope = nullptr;                       // distance slopes [heads]
     float* d_conv = nullptr;                        // weights of the convolution behind the projections [q channels | k channels][taps]
     float rot_amp = 1.0f;                           // factor on cos and sin of the rotation
+    // recurrent mixers
+    int i_off = 0, f_off = 0;                       // gate pre-activations (input / forget; decay / beta)
+    float *d_Alog = nullptr, *d_dtb = nullptr, *d_D = nullptr, *d_cbias = nullptr;
+    bf16 *w_x = nullptr, *w_dt = nullptr;           // selective scan: input-dependent projections
+    int ld_x = 0, ld_bc = 0, dt_p = 0;
+    float* d_join = nullptr;                        // weight of the norm behind this branch's own out projection
+    int ko_p = 0;                                   // K of that projection
 };
 
 struct LayerW {
@@ -115,6 +123,7 @@ struct Run {
     bool enters_pass = false;  // the loop's entry projection comes before this run
     void *kc[2] = {nullptr, nullptr}, *vc[2] = {nullptr, nullptr};
     float* state[2] = {nullptr, nullptr};
+    float* mstate[2] = {nullptr, nullptr};  // mLSTM: running maximum of the log gates [n_slots][heads]
     float* tail = nullptr;
     float* ctail = nullptr;                 // last taps - 1 projected values of the convolution behind the projections [n_slots][taps - 1][channels]
     int ctail_n = 0;                        // floats per slot
@@ -143,6 +152,16 @@ struct gtb_seq_model {
     float* qk_sc = nullptr;                      // scales of the whole-projection q / k norm [max_rows][2]
     float *xs = nullptr, *hc_one = nullptr, *latQ = nullptr, *latQA = nullptr, *Y2 = nullptr, *shw = nullptr;
     void *opQ = nullptr, *opO = nullptr;
+    // recurrent mixers
+    float4* recG = nullptr;                      // gates of a pass [max_rows][heads]
+    float2* recB = nullptr;                      // running sums of the log decays inside a chunk
+    int rec_heads_max = 0;
+    bf16 *recQ = nullptr, *recK = nullptr, *recW = nullptr, *recV = nullptr, *recS = nullptr;    // planes: q, k, W, values / u, states before the chunks
+    size_t rec_qk_max = 0, rec_w_max = 0, rec_v_max = 0, rec_s_max = 0;     // elements per plane (recS: elements)
+    float *ssmBC = nullptr, *ssmDT = nullptr;    // selective scan: [step rank | B | C] and step sizes of a pass
+    void *opX = nullptr, *opDT = nullptr;
+    int ssm_bc_max = 0, ssm_inner_max = 0, ssm_x_max = 0, ssm_dt_max = 0;
+    bool join = false;
     float* latX = nullptr;                       // expanded [plain keys | values] of one segment's visible range, fp32 [max_ctx][heads * (dim + vdim)]
     bf16 *latKx = nullptr, *latVx = nullptr;     // the same as bf16 heads [n_slots][max_ctx][heads][dim + rope | vdim], shared by the layers
     int lat_kx_max = 0, lat_vx_max = 0, lat_x_max = 0;
@@ -257,7 +276,15 @@ int upload_rot_table(gtb_seq_model* m, BranchW& b) {
     return GTB_OK;
 }
 // fp32 values of recurrent state one slot holds for a branch
-size_t state_floats(const gtb_seq_branch& d) { return d.kind == GTB_MIX_MINGRU ? (size_t)d.dim : (size_t)d.heads * d.dim * d.vdim; }
+bool rec_kind(int kind) { return kind == GTB_MIX_MLSTM || kind == GTB_MIX_DELTA; }
+int rec_vx(const gtb_seq_branch& d) { return d.vdim + (d.kind == GTB_MIX_MLSTM ? 1 : 0); }
+size_t state_floats(const gtb_seq_branch& d) {
+    if (rec_kind(d.kind)) return (size_t)d.heads * d.dim * ((rec_vx(d) + 3) & ~3);
+    if (d.kind == GTB_MIX_SSM) return (size_t)d.inner * d.state;
+    return d.kind == GTB_MIX_MINGRU ? (size_t)d.dim : (size_t)d.heads * d.dim * d.vdim;
+}
+// chunked mLSTM / delta rule (prompt portions, bf16 mode): rows per chunk, or 0 when the head is too wide for the chunk kernels' shared memory
+int rec_chunk(const gtb_seq_branch& d) { return d.dim <= 128 ? 64 : d.dim <= 256 ? 32 : 0; }
 constexpr int GRU_CHUNK = 32;               // rows per chunk of the chunked minGRU scan
 
 // C = (acc ? C : 0) + bias + A . W^T on the library stream; picks the tensor-core kernel, the few-row kernel or the SIMT tile kernel
@@ -572,11 +599,17 @@ NormArgs sw_norm(const gtb_seq_model* m, const LayerW& l, int q) {          // q
 // the residual update with the fewest kept values per thread that hold a row of this width
 template <typename OT>
 void sandwich_add(int R, size_t smem, const float* Y, const float* Y2, const float* Yg, const int* pair_dst, int top, int W, const NormArgs& post, float* x, const NormArgs& next,
-                  OT* op, int ld_op, const GroupRouteNext& rn) {
+                  OT* op, int ld_op, const GroupRouteNext& rn, const JoinArgs* jn = nullptr) {
     cudaStream_t st = ctx().stream;
-    if (W <= 1024) k_sandwich_add<OT, 1><<<R, 256, smem, st>>>(Y, Y2, Yg, pair_dst, top, W, post, x, next, op, ld_op, rn);
-    else if (W <= 2048) k_sandwich_add<OT, 2><<<R, 256, smem, st>>>(Y, Y2, Yg, pair_dst, top, W, post, x, next, op, ld_op, rn);
-    else k_sandwich_add<OT, 4><<<R, 256, smem, st>>>(Y, Y2, Yg, pair_dst, top, W, post, x, next, op, ld_op, rn);
+    if (jn) {
+        if (W <= 1024) k_sandwich_add<OT, 1, true><<<R, 256, smem, st>>>(Y, Y2, Yg, pair_dst, top, W, post, x, next, op, ld_op, rn, *jn);
+        else if (W <= 2048) k_sandwich_add<OT, 2, true><<<R, 256, smem, st>>>(Y, Y2, Yg, pair_dst, top, W, post, x, next, op, ld_op, rn, *jn);
+        else k_sandwich_add<OT, 4, true><<<R, 256, smem, st>>>(Y, Y2, Yg, pair_dst, top, W, post, x, next, op, ld_op, rn, *jn);
+        return;
+    }
+    if (W <= 1024) k_sandwich_add<OT, 1><<<R, 256, smem, st>>>(Y, Y2, Yg, pair_dst, top, W, post, x, next, op, ld_op, rn, JoinArgs{});
+    else if (W <= 2048) k_sandwich_add<OT, 2><<<R, 256, smem, st>>>(Y, Y2, Yg, pair_dst, top, W, post, x, next, op, ld_op, rn, JoinArgs{});
+    else k_sandwich_add<OT, 4><<<R, 256, smem, st>>>(Y, Y2, Yg, pair_dst, top, W, post, x, next, op, ld_op, rn, JoinArgs{});
 }
 
 // The convolution behind the q and k projections of a softmax-attention branch: convolved queries to m->convQ, keys (and plain values) to the
@@ -676,6 +709,156 @@ int run_soft_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const R
         GTB_LAUNCHED();
     }
     return GTB_OK;
+}
+
+// ---- recurrent mixers with token-dependent decays ------------------------------------------------------------------------------
+// causal convolution (and silu) of `nq` projected columns from `off` on into m->convQ, the slots' histories brought up to date
+template <typename OT>
+int run_act_conv(gtb_seq_model* m, const PassTables& t, int R, int S, const Run& run, const BranchW& b, const LayerW& l, int off, int nq, void* op, int ld_op) {
+    ConvArgs a{};
+    a.nq = nq; a.off = off; a.taps = b.d.conv; a.w = b.d_conv; a.max_ctx = m->cfg.max_ctx; a.bias = b.d_cbias; a.silu = 1; a.op = op; a.ld_op = ld_op;
+    const bool vec = ((nq | off | l.n1) & 3) == 0;
+    const int rows_per = R >= 512 ? 16 : R >= 64 ? 4 : 1, every_one = R == S && a.taps <= 4;
+    if (vec) launch_qk_conv<OT, 4>(t, a, m->P, l.n1, R, rows_per, run.ctail, m->convQ, (OT*)nullptr, (OT*)nullptr, every_one);
+    else launch_qk_conv<OT, 1>(t, a, m->P, l.n1, R, rows_per, run.ctail, m->convQ, (OT*)nullptr, (OT*)nullptr, every_one);
+    GTB_LAUNCHED();
+    if (a.taps > 1 && !every_one) {
+        k_canon_tail<<<dim3(S, (nq + 255) / 256), 256, 0, ctx().stream>>>(t, m->P + off, l.n1, nq, a.taps, run.ctail);
+        GTB_LAUNCHED();
+    }
+    return GTB_OK;
+}
+
+RecBranch rec_args(const gtb_seq_model* m, const BranchW& b) {
+    RecBranch a{};
+    a.heads = b.d.heads; a.kv_heads = b.d.kv_heads; a.dim = b.d.dim; a.vdim = b.d.vdim;
+    a.vx = rec_vx(b.d); a.vxp = (a.vx + 3) & ~3; a.dp = (a.dim + 15) & ~15; a.vp = (a.vx + 15) & ~15;
+    a.cap = b.d.gate_cap; a.eps = m->cfg.eps; a.qscale = b.d.scale; a.out_scale = b.d.out_scale;
+    a.q_off = b.q_off; a.k_off = b.k_off; a.v_off = b.v_off; a.i_off = b.i_off; a.f_off = b.f_off; a.g_off = b.g_off; a.a_off = b.a_off;
+    a.A_log = b.d_Alog; a.dt_bias = b.d_dtb; a.norm = b.d_onorm;
+    return a;
+}
+
+template <int KIND>
+int launch_rec_walk(const PassTables& t, const RecBranch& a, int S, const float* X, int ldx, const float4* G, float* state, float* O) {
+    const dim3 grid(S, a.heads, (a.vx + 31) / 32);
+    cudaStream_t st = ctx().stream;
+    if (a.dim <= 32) k_rec_walk<KIND, 4><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
+    else if (a.dim <= 64) k_rec_walk<KIND, 8><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
+    else if (a.dim <= 128) k_rec_walk<KIND, 16><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
+    else if (a.dim <= 256) k_rec_walk<KIND, 32><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
+    else if (a.dim <= 512) k_rec_walk<KIND, 64><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
+    else k_rec_walk<KIND, 128><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
+    GTB_LAUNCHED();
+    return GTB_OK;
+}
+template <int KIND, int C, int MT>
+int launch_rec_scan(gtb_seq_model* m, const PassTables& t, const RecBranch& a, int S, size_t ps_qk, size_t ps_w, size_t ps_v, const float* X, int ldx, float* state) {
+    const size_t smem = ((size_t)(KIND == REC_DELTA ? 8 : 4) * C * (a.dp + 8) + 2 * (size_t)a.dp * (REC_VS + 8) + 2 * C * (REC_VS + 8)) * 2;
+    static size_t allowed = 48 * 1024;
+    if (smem > allowed) { GTB_CUDA(cudaFuncSetAttribute(k_rec_scan<KIND, C, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); allowed = smem; }
+    k_rec_scan<KIND, C, MT><<<dim3(S, a.heads, a.vp / REC_VS), 256, smem, ctx().stream>>>(t, a, m->recK, ps_qk, m->recW, ps_w, m->recG, m->recB, X, ldx, m->recV, ps_v, m->recS, state);
+    GTB_LAUNCHED();
+    return GTB_OK;
+}
+template <int VP, int C>
+int launch_rec_out(gtb_seq_model* m, const PassTables& t, const RecBranch& a, int kind, int S, int n_chunks, size_t ps_qk, size_t ps_v) {
+    const size_t smem = (4 * (size_t)C * 72 + 2 * 64 * (size_t)(VP + 8)) * 2;
+    static bool attr = false;
+    if (!attr) { GTB_CUDA(cudaFuncSetAttribute(k_rec_out<VP, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); attr = true; }
+    k_rec_out<VP, C><<<dim3(n_chunks, a.heads, (a.vp + VP - 1) / VP), 2 * C, smem, ctx().stream>>>(t, a, kind, S, m->recQ, m->recK, ps_qk, m->recV, ps_v, m->recS, m->recG, m->recB, m->O);
+    GTB_LAUNCHED();
+    return GTB_OK;
+}
+template <int KIND, int C>
+int run_rec_chunks(gtb_seq_model* m, const PassTables& t, const RecBranch& a, int R, int S, int n_chunks, float* X, int ldx, float* state) {
+    cudaStream_t st = ctx().stream;
+    const size_t ps_qk = (size_t)m->max_rows * a.kv_heads * a.dp, ps_w = (size_t)m->max_rows * a.heads * a.dp, ps_v = (size_t)m->max_rows * a.heads * a.vp;
+    const int units = 2 * a.kv_heads + (KIND == REC_MLSTM ? a.heads : 0);
+    k_rec_prep<KIND><<<dim3(R, (units + 7) / 8), 256, 0, st>>>(a, X, ldx, m->recQ, m->recK, ps_qk, m->recV, ps_v);
+    GTB_LAUNCHED();
+    if (KIND == REC_DELTA) {
+        const size_t smem = (size_t)C * (C + 4) * sizeof(float) + 2 * (size_t)C * (a.dp + 8) * 2;
+        static size_t allowed = 48 * 1024;
+        if (smem > allowed) { GTB_CUDA(cudaFuncSetAttribute(k_delta_wy<C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); allowed = smem; }
+        k_delta_wy<C><<<dim3(n_chunks, a.heads), 256, smem, st>>>(t, a, S, m->recK, ps_qk, m->recG, m->recB, X, ldx, m->recW, ps_w);
+        GTB_LAUNCHED();
+    }
+    int rc = a.dp <= 128 ? launch_rec_scan<KIND, C, 1>(m, t, a, S, ps_qk, ps_w, ps_v, X, ldx, state) : launch_rec_scan<KIND, C, 2>(m, t, a, S, ps_qk, ps_w, ps_v, X, ldx, state);
+    if (rc) return rc;
+    if (a.vp <= 32) return launch_rec_out<32, C>(m, t, a, KIND, S, n_chunks, ps_qk, ps_v);
+    if (a.vp <= 64 || a.vp % 64 == 0) return launch_rec_out<64, C>(m, t, a, KIND, S, n_chunks, ps_qk, ps_v);
+    return launch_rec_out<80, C>(m, t, a, KIND, S, n_chunks, ps_qk, ps_v);
+}
+
+// One mLSTM or delta-rule branch on R rows: projections in m->P, gated output into the out-projection operand.
+template <typename OT, int KIND>
+int run_rec_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const Run& run, int bi, const LayerW& l, bool portions, const int* seg_lens) {
+    cudaStream_t st = ctx().stream;
+    const BranchW& b = l.br[bi];
+    RecBranch a = rec_args(m, b);
+    float* X = m->P;
+    int ldx = l.n1;
+    if (KIND == REC_DELTA) {
+        const int nq = b.kq + b.kk + b.kv;
+        int rc = run_act_conv<OT>(m, t, R, S, run, b, l, b.q_off, nq, nullptr, 0);
+        if (rc) return rc;
+        X = m->convQ; ldx = nq;
+        a.q_off = 0; a.k_off = b.kq; a.v_off = b.kq + b.kk;
+    }
+    const int C = rec_chunk(b.d);
+    const bool chunks = sizeof(OT) == 2 && portions && C > 0;
+    k_rec_gates<KIND><<<dim3(S, a.heads), R == S ? 32 : chunks || R >= 64 * S ? 512 : 64, 0, st>>>(t, a, m->P, l.n1, C, run.mstate[bi], m->recG, chunks ? m->recB : nullptr);
+    GTB_LAUNCHED();
+    int rc;
+    if (chunks) {
+        int n_chunks = 0;
+        for (int s = 0; s < S; s++) n_chunks += (seg_lens[s] + C - 1) / C;
+        if ((size_t)n_chunks * a.heads * 2 * a.dp * a.vp > m->rec_s_max) return gtb::fail(GTB_ERR_STATE, "chunk workspace too small");
+        rc = C == 64 ? run_rec_chunks<KIND, 64>(m, t, a, R, S, n_chunks, X, ldx, run.state[bi]) : run_rec_chunks<KIND, 32>(m, t, a, R, S, n_chunks, X, ldx, run.state[bi]);
+    } else {
+        if (KIND == REC_DELTA) {
+            k_rec_unit<<<dim3(R, (2 * a.kv_heads + 3) / 4), 128, 0, st>>>(a, X, ldx);
+            GTB_LAUNCHED();
+        }
+        rc = launch_rec_walk<KIND>(t, a, S, X, ldx, m->recG, run.state[bi], m->O);
+    }
+    if (rc) return rc;
+    k_rec_post<OT, KIND><<<dim3(R, (a.heads + 3) / 4), 128, 0, st>>>(a, m->O, m->recG, m->P, l.n1, (OT*)m->opC, l.kout_p);
+    GTB_LAUNCHED();
+    return GTB_OK;
+}
+
+template <typename OT, int LANES, int KS>
+int launch_ssm(const PassTables& t, const SsmBranch& a, int S, const float* XC, const float* DT, const float* BC, int ld_bc, const float* P, int ldp, float* state, OT* out, int ld_out) {
+    constexpr int NCH = 128 / LANES;
+    k_ssm_scan<OT, LANES, KS><<<dim3(S, (a.inner + NCH - 1) / NCH), 128, 0, ctx().stream>>>(t, a, XC, DT, BC, ld_bc, P, ldp, state, out, ld_out);
+    GTB_LAUNCHED();
+    return GTB_OK;
+}
+// One selective-scan branch on R rows: projections in m->P, gated output into the out-projection operand.
+template <typename OT>
+int run_ssm_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const Run& run, int bi, const LayerW& l) {
+    cudaStream_t st = ctx().stream;
+    const BranchW& b = l.br[bi];
+    SsmBranch a{};
+    a.inner = b.d.inner; a.state = b.d.state; a.dt_rank = b.d.dt_rank; a.z_off = b.q_off + b.d.inner; a.a_off = b.a_off; a.A_log = b.d_Alog; a.D = b.d_D; a.out_scale = b.d.out_scale;
+    int rc = run_act_conv<OT>(m, t, R, S, run, b, l, b.q_off, a.inner, m->opX, b.ld_x);
+    if (rc) return rc;
+    const int nbc = a.dt_rank + 2 * a.state;
+    rc = product<OT>(m, m->opX, b.ld_x, b.w_x, b.ld_x, m->ssmBC, b.ld_bc, R, nbc, b.ld_x, nullptr, 0);
+    if (rc) return rc;
+    if (sizeof(OT) == 2 && m->use_tensor && m->gp && R >= m->tensor_min_rows) {
+        k_cols_operand<OT><<<R, 64, 0, st>>>(m->ssmBC, b.ld_bc, a.dt_rank, (OT*)m->opDT, b.dt_p);
+        GTB_LAUNCHED();
+        rc = product<OT>(m, m->opDT, b.dt_p, b.w_dt, b.dt_p, m->ssmDT, a.inner, R, a.inner, b.dt_p, b.d_dtb, 0);
+    } else rc = product<float>(m, m->ssmBC, b.ld_bc, b.w_dt, b.dt_p, m->ssmDT, a.inner, R, a.inner, b.dt_p, b.d_dtb, 0);    // (the columns behind dt_rank meet zero weights)
+    if (rc) return rc;
+    OT* out = (OT*)m->opC;
+#define SSM_CASE(N, LN, KS) if (a.state <= N) return launch_ssm<OT, LN, KS>(t, a, S, m->convQ, m->ssmDT, m->ssmBC, b.ld_bc, m->P, l.n1, run.state[bi], out, l.kout_p)
+    SSM_CASE(4, 1, 4); SSM_CASE(8, 2, 4); SSM_CASE(16, 4, 4); SSM_CASE(32, 8, 4); SSM_CASE(64, 16, 4); SSM_CASE(128, 32, 4); SSM_CASE(256, 32, 8);
+#undef SSM_CASE
+    return gtb::fail(GTB_ERR_STATE, "selective scan of %d states per channel", a.state);
 }
 
 // ---- latent attention (pre-norm and sandwich layers) ---------------------------------------------------------------------------
@@ -800,6 +983,68 @@ int run_latent_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const
     return GTB_OK;
 }
 
+// where the output of a layer's gated experts is: one row per row in Y, or rows pair_dst[r * top + k] of Yg to be summed; Y2: the shared expert's share
+struct ExpertOut {
+    const float *Y = nullptr, *Y2 = nullptr, *Yg = nullptr;
+    const int* pair_dst = nullptr;
+    int top = 0;
+};
+// Gated routed experts on R rows of opA (pre-norm and sandwich layers).  is_routed: the choices are in sel_idx / sel_w already.
+template <typename OT>
+int run_gated_experts(gtb_seq_model* m, int R, const LayerW& l, bool is_routed, ExpertOut& eo) {
+    cudaStream_t st = ctx().stream;
+    const int W = m->cfg.width, wp = m->wp, E = l.d.experts, top = l.d.top;
+    OT *opA = (OT*)m->opA, *opC = (OT*)m->opC;
+    int rc;
+    if (!is_routed) {                        // router (and the shared expert's gate) in one product, fp32 accumulation
+        rc = product<OT>(m, opA, wp, l.w_router, wp, m->rl, l.n_out, R, l.n_out, wp, nullptr, 0);
+        if (rc) return rc;
+        if (l.d.route_kind == GTB_ROUTE_SOFTMAX) k_moe_route_softmax<<<R, 32, E * sizeof(float), st>>>(m->rl, l.n_out, E, top, m->sel_idx, m->sel_w);
+        else k_moe_route_sigmoid<<<R, 32, E * sizeof(float), st>>>(m->rl, l.n_out, E, top, m->sel_idx, m->sel_w, l.sff > 0 ? m->shw : nullptr);
+        GTB_LAUNCHED();
+    }
+    if (l.sff > 0) {
+        bool act_done = false;
+        if (sizeof(OT) == 2 && m->use_tensor && m->gp && R >= m->tensor_min_rows && l.sh_inter) {
+            rc = seq_gemm_bf16_gated(m->gp, opA, wp, l.w_sh_gu, wp, opC, l.sff_p, 0, R, 2 * l.sff, wp, 1, m->shw);
+            if (rc > 0) return rc;
+            if (rc == 0) { ctx().launches++; act_done = true; }
+        }
+        if (!act_done) {
+            rc = product<OT>(m, opA, wp, l.w_sh_gu, wp, m->G, 2 * l.sff, R, 2 * l.sff, wp, nullptr, 0);
+            if (rc) return rc;
+            k_swiglu_rows<OT><<<dim3(R, std::max(1, std::min((l.sff_p + 255) / 256, std::max(1, 2048 / R)))), 256, 0, st>>>(m->G, l.sff, l.sh_inter ? 1 : 0, m->shw, opC, l.sff_p);
+            GTB_LAUNCHED();
+        }
+        rc = product<OT>(m, opC, l.sff_p, l.w_sh_down, l.sff_p, m->Y2, W, R, W, l.sff_p, nullptr, 0);
+        if (rc) return rc;
+        eo.Y2 = m->Y2;
+    }
+    const int n_pairs = R * top, mpad = (n_pairs + 127) / 128 * 128 + E * 128;
+    if (sizeof(OT) == 2 && m->grouped_experts && m->use_tensor && m->gp && m->Xg && l.e_inter && R >= m->tensor_min_rows && mpad <= m->mpad_max) {
+        // rows sorted by expert; the gate-and-up product writes w * silu(gate) * up per (row, choice), the down product one output row per pair,
+        // and the residual update sums a row's pairs
+        k_moe_group<<<1, 1024, 2 * E * sizeof(int), st>>>(m->sel_idx, n_pairs, E, m->pair_dst, m->tile_e, mpad / 128);
+        GTB_LAUNCHED();
+        k_moe_gather<<<n_pairs, 128, 0, st>>>((const bf16*)opA, wp, top, m->pair_dst, m->sel_w, m->Xg, m->rw);
+        GTB_LAUNCHED();
+        rc = seq_gemm_bf16_grouped_gated(m->gp, m->Xg, wp, l.w_up, wp, mpad, 2 * l.ff, wp, E, m->tile_e, m->actg, l.kfp, m->rw, 1);
+        if (rc == 0) rc = seq_gemm_bf16_grouped(m->gp, m->actg, l.kfp, l.w_down, l.kfp, mpad, W, l.kfp, E, m->tile_e, m->Yg, W, nullptr, 0, nullptr);
+        if (rc > 0) return rc;
+        if (rc == 0) {
+            eo.Yg = m->Yg; eo.pair_dst = m->pair_dst; eo.top = top;
+            return GTB_OK;
+        }
+    }
+    const int cta_budget = std::max(1, 4096 / std::max(1, R * top));
+    k_moe_gu_rows<OT><<<dim3(R * top, std::max(1, std::min(cta_budget, (l.kfp + 7) / 8))), 256, 0, st>>>(opA, wp, wp, l.w_up, wp, l.ff, l.kfp, l.e_inter ? 1 : 0, top, m->sel_idx, m->sel_w, (OT*)m->act);
+    GTB_LAUNCHED();
+    k_moe_down_rows<OT><<<dim3(R, std::max(1, std::min(std::max(1, 4096 / R), (W + 7) / 8))), 256, 0, st>>>((const OT*)m->act, l.kfp, l.w_down, W, E, top, m->sel_idx, m->Y, W);
+    GTB_LAUNCHED();
+    eo.Y = m->Y;
+    return GTB_OK;
+}
+
 // One layer of the sandwich style on R rows: x += norm1b(mixer(norm1(x))); x += norm2b(ff(norm2(x))).  opA holds norm1(x) on entry; on
 // return it holds `next` of the new stream (the following layer's norm1) when next.w is set.
 template <typename OT>
@@ -814,24 +1059,46 @@ int run_sandwich_layer(gtb_seq_model* m, const PassTables& t, int R, int S, cons
     for (int bi = 0; bi < l.d.n_branches; bi++) {
         if (l.br[bi].d.kind == GTB_MIX_SOFTMAX_ATTN) rc = run_soft_branch<OT>(m, t, R, S, run, bi, l, portions, n_qtiles);
         else if (l.br[bi].d.kind == GTB_MIX_LATENT_ATTN) rc = run_latent_branch<OT>(m, t, R, S, run, l, portions, seg_lens, seg_slots, n_qtiles);
+        else if (l.br[bi].d.kind == GTB_MIX_MLSTM) rc = run_rec_branch<OT, REC_MLSTM>(m, t, R, S, run, bi, l, portions, seg_lens);
+        else if (l.br[bi].d.kind == GTB_MIX_DELTA) rc = run_rec_branch<OT, REC_DELTA>(m, t, R, S, run, bi, l, portions, seg_lens);
+        else if (l.br[bi].d.kind == GTB_MIX_SSM) rc = run_ssm_branch<OT>(m, t, R, S, run, bi, l);
         else rc = run_retention<OT>(m, t, R, S, run, bi, l, portions, seg_lens);
         if (rc) return rc;
     }
-    rc = product<OT>(m, opC, l.kout_p, l.w_out, l.kout_p, m->Y, W, R, W, l.kout_p, l.d_obias, 0);
+    JoinArgs jn{};
+    if (l.d.join_norm) {                     // two out projections, joined in the residual update
+        for (int bi = 0; bi < 2; bi++) {
+            const BranchW& b = l.br[bi];
+            rc = product<OT>(m, opC + b.a_off, l.kout_p, l.w_out + b.a_off, l.kout_p, bi ? m->Y2 : m->Y, W, R, W, b.ko_p, nullptr, 0);
+            if (rc) return rc;
+        }
+        jn.w1 = l.br[0].d_join; jn.w2 = l.br[1].d_join; jn.scale = 0.5f; jn.eps = c.eps;
+    } else rc = product<OT>(m, opC, l.kout_p, l.w_out, l.kout_p, m->Y, W, R, W, l.kout_p, l.d_obias, 0);
     if (rc) return rc;
     // few rows and a routed feed-forward next: the residual update also computes the router's logits from the operand row it has just formed
     // and picks the experts (two launches less per layer on a decode step)
     GroupRouteNext rn{};
     const int groups = std::max(1, l.d.route_groups), keep = l.d.route_keep > 0 ? l.d.route_keep : groups;
-    const bool routed = l.ff > 0 && l.d.ff_kind == GTB_FF_GROUP_EXPERTS;
+    const bool gated_moe = l.ff > 0 && l.d.ff_kind == GTB_FF_GATED_EXPERTS;
+    const bool routed = (l.ff > 0 && l.d.ff_kind == GTB_FF_GROUP_EXPERTS) || (gated_moe && l.d.route_kind == GTB_ROUTE_SOFTMAX && l.sff == 0);
     const size_t rn_smem = routed ? ((size_t)W + 3 * l.d.experts + groups) * sizeof(float) : 0;
     if (routed && R <= 8 && rn_smem <= 40 * 1024) {
+        rn.kind = gated_moe ? 1 : 0;
         rn.w = l.w_router; rn.ldw = wp; rn.n_exp = l.d.experts; rn.n_groups = groups; rn.keep = keep; rn.top = l.d.top; rn.n_always = l.n_sh; rn.scale = l.d.route_scale;
         rn.sel_idx = m->sel_idx; rn.sel_w = m->sel_w;
     }
-    sandwich_add<OT>(R, rn.w ? rn_smem : 0, m->Y, nullptr, nullptr, nullptr, 0, W, sw_norm(m, l, 1), m->x, l.ff > 0 ? sw_norm(m, l, 2) : next, opA, wp, rn);
+    sandwich_add<OT>(R, rn.w ? rn_smem : 0, m->Y, l.d.join_norm ? m->Y2 : nullptr, nullptr, nullptr, 0, W, sw_norm(m, l, 1), m->x, l.ff > 0 ? sw_norm(m, l, 2) : next, opA, wp, rn,
+                     l.d.join_norm ? &jn : nullptr);
     GTB_LAUNCHED();
     if (l.ff == 0) return GTB_OK;
+    if (gated_moe) {
+        ExpertOut eo;
+        rc = run_gated_experts<OT>(m, R, l, rn.w != nullptr, eo);
+        if (rc) return rc;
+        sandwich_add<OT>(R, 0, eo.Y, eo.Y2, eo.Yg, eo.pair_dst, eo.top, W, sw_norm(m, l, 3), m->x, next, opA, wp, GroupRouteNext{});
+        GTB_LAUNCHED();
+        return GTB_OK;
+    }
     if (l.d.ff_kind == GTB_FF_GELU) {
         bool act_done = false;
         if (sizeof(OT) == 2 && m->use_tensor && m->gp && R >= m->tensor_min_rows) {
@@ -984,53 +1251,10 @@ int run_prenorm_layer(gtb_seq_model* m, const PassTables& t, int R, int S, const
         pend.Y = m->Y; pend.hc = l.hc[1];
         return GTB_OK;
     }
-    // gated routed experts: router (and the shared expert's gate) in one product, fp32 accumulation
-    const int E = l.d.experts, top = l.d.top;
-    rc = product<OT>(m, opA, wp, l.w_router, wp, m->rl, l.n_out, R, l.n_out, wp, nullptr, 0);
+    ExpertOut eo;
+    rc = run_gated_experts<OT>(m, R, l, false, eo);
     if (rc) return rc;
-    k_moe_route_sigmoid<<<R, 32, E * sizeof(float), st>>>(m->rl, l.n_out, E, top, m->sel_idx, m->sel_w, l.sff > 0 ? m->shw : nullptr);
-    GTB_LAUNCHED();
-    if (l.sff > 0) {
-        bool act_done = false;
-        if (sizeof(OT) == 2 && m->use_tensor && m->gp && R >= m->tensor_min_rows && l.sh_inter) {
-            rc = seq_gemm_bf16_gated(m->gp, opA, wp, l.w_sh_gu, wp, opC, l.sff_p, 0, R, 2 * l.sff, wp, 1, m->shw);
-            if (rc > 0) return rc;
-            if (rc == 0) { ctx().launches++; act_done = true; }
-        }
-        if (!act_done) {
-            rc = product<OT>(m, opA, wp, l.w_sh_gu, wp, m->G, 2 * l.sff, R, 2 * l.sff, wp, nullptr, 0);
-            if (rc) return rc;
-            k_swiglu_rows<OT><<<dim3(R, std::max(1, std::min((l.sff_p + 255) / 256, std::max(1, 2048 / R)))), 256, 0, st>>>(m->G, l.sff, l.sh_inter ? 1 : 0, m->shw, opC, l.sff_p);
-            GTB_LAUNCHED();
-        }
-        rc = product<OT>(m, opC, l.sff_p, l.w_sh_down, l.sff_p, m->Y2, W, R, W, l.sff_p, nullptr, 0);
-        if (rc) return rc;
-        pend.Y2 = m->Y2;
-    }
-    const int n_pairs = R * top, mpad = (n_pairs + 127) / 128 * 128 + E * 128;
-    if (sizeof(OT) == 2 && m->grouped_experts && m->use_tensor && m->gp && m->Xg && l.e_inter && R >= m->tensor_min_rows && mpad <= m->mpad_max) {
-        // rows sorted by expert; the gate-and-up product writes w * silu(gate) * up per (row, choice), the down product one output row per pair,
-        // and the next boundary sums a row's pairs
-        k_moe_group<<<1, 1024, 2 * E * sizeof(int), st>>>(m->sel_idx, n_pairs, E, m->pair_dst, m->tile_e, mpad / 128);
-        GTB_LAUNCHED();
-        k_moe_gather<<<n_pairs, 128, 0, st>>>((const bf16*)opA, wp, top, m->pair_dst, m->sel_w, m->Xg, m->rw);
-        GTB_LAUNCHED();
-        rc = seq_gemm_bf16_grouped_gated(m->gp, m->Xg, wp, l.w_up, wp, mpad, 2 * l.ff, wp, E, m->tile_e, m->actg, l.kfp, m->rw, 1);
-        if (rc == 0) rc = seq_gemm_bf16_grouped(m->gp, m->actg, l.kfp, l.w_down, l.kfp, mpad, W, l.kfp, E, m->tile_e, m->Yg, W, nullptr, 0, nullptr);
-        if (rc > 0) return rc;
-        if (rc == 0) {
-            pend.Yg = m->Yg; pend.pair_dst = m->pair_dst; pend.top = top; pend.hc = l.hc[1];
-            return GTB_OK;
-        }
-    }
-    {
-        const int cta_budget = std::max(1, 4096 / std::max(1, R * top));
-        k_moe_gu_rows<OT><<<dim3(R * top, std::max(1, std::min(cta_budget, (l.kfp + 7) / 8))), 256, 0, st>>>(opA, wp, wp, l.w_up, wp, l.ff, l.kfp, l.e_inter ? 1 : 0, top, m->sel_idx, m->sel_w, (OT*)m->act);
-        GTB_LAUNCHED();
-        k_moe_down_rows<OT><<<dim3(R, std::max(1, std::min(std::max(1, 4096 / R), (W + 7) / 8))), 256, 0, st>>>((const OT*)m->act, l.kfp, l.w_down, W, E, top, m->sel_idx, m->Y, W);
-        GTB_LAUNCHED();
-    }
-    pend.Y = m->Y; pend.hc = l.hc[1];
+    pend.Y = eo.Y; pend.Y2 = eo.Y2; pend.Yg = eo.Yg; pend.pair_dst = eo.pair_dst; pend.top = eo.top; pend.hc = l.hc[1];
     return GTB_OK;
 }
 
@@ -1187,7 +1411,8 @@ int run_pass(gtb_seq_model* m, const PassTables& t, int R, int S, bool from_pend
     }
     if (n_want > 0) {
         float ls = c.logit_scale != 0.0f ? c.logit_scale : 1.0f;        // what is left of the logit scale for the logits themselves
-        if (c.final_norm >= 3) {
+        if (c.final_norm == 5) k_rmsnorm_weight<OT><<<n_want, 256, 0, st>>>(m->x, W, c.eps, m->final_gain, 0, d_want, opH, wp);
+        else if (c.final_norm >= 3) {
             NormArgs fn{};
             fn.kind = GTB_NORM_LAYER; fn.w = m->final_gain; fn.b = m->final_b; fn.eps = c.eps;
             k_norm_rows<OT><<<n_want, 256, 0, st>>>(m->x, W, fn, d_want, opH, wp, ls);      // the product is linear: the scale rides on its operand
@@ -1209,6 +1434,52 @@ int run_pass(gtb_seq_model* m, const PassTables& t, int R, int S, bool from_pend
     }
     k_commit<<<(S + 127) / 128, 128, 0, st>>>(t, S);
     GTB_LAUNCHED();
+    return GTB_OK;
+}
+
+// tensors of a layer's gated routed experts (and the shared expert)
+int want_gated_experts(gtb_seq_model* m, LayerW& l, const std::string& lp) {
+    const int W = m->cfg.width, wp = m->wp;
+    int rc = GTB_OK;
+#define TRY(e) do { rc = (e); if (rc) return rc; } while (0)
+#define REQ(cond) do { if (!(cond)) return gtb::fail(GTB_ERR_ARG, "model description rejected: %s", #cond); } while (0)
+    const int E = l.d.experts;
+    REQ(E > 0 && E <= 4096 && l.d.identity == 0 && l.d.top > 0 && l.d.top <= E && l.d.top <= 64 && l.d.shared_ff >= 0);
+    l.sff = l.d.shared_ff;
+    l.n_out = E + (l.sff > 0 ? 1 : 0);
+    TRY(dalloc_t(m, &l.w_router, (size_t)l.n_out * wp));
+    want_matrix(m, lp + "mlp.router", l.w_router, E, W, wp);
+    if (l.sff > 0) want_matrix(m, lp + "mlp.shared.sg", l.w_router + (size_t)E * wp, 1, W, wp);
+    TRY(dalloc_t(m, &l.w_up, (size_t)E * 2 * l.ff * wp));
+    TRY(dalloc_t(m, &l.w_down, (size_t)E * W * l.kfp));
+    l.e_inter = l.ff % 32 == 0;
+    for (int e = 0; e < E; e++) {
+        const std::string ep = lp + "mlp.e" + std::to_string(e) + ".";
+        bf16* base = l.w_up + (size_t)e * 2 * l.ff * wp;
+        want_matrix(m, ep + "gate", base, l.ff, W, wp);
+        want_matrix(m, ep + "up", base + (size_t)(l.e_inter ? 32 : l.ff) * wp, l.ff, W, wp);
+        if (l.e_inter)
+            for (const char* nm : {"gate", "up"}) { TensorDest& d = m->tensors[ep + nm]; d.group = 32; d.group_stride = 64; }
+        want_matrix(m, ep + "down", l.w_down + (size_t)e * W * l.kfp, W, l.ff, l.kfp);
+    }
+    m->n_out_max = std::max(m->n_out_max, l.n_out);
+    m->top_max = std::max(m->top_max, l.d.top);
+    m->e_max = std::max(m->e_max, E);
+    if (l.sff > 0) {
+        l.sff_p = pad64(l.sff);
+        l.sh_inter = l.sff % 32 == 0;
+        TRY(dalloc_t(m, &l.w_sh_gu, (size_t)2 * l.sff * wp));
+        TRY(dalloc_t(m, &l.w_sh_down, (size_t)W * l.sff_p));
+        want_matrix(m, lp + "mlp.shared.gate", l.w_sh_gu, l.sff, W, wp);
+        want_matrix(m, lp + "mlp.shared.up", l.w_sh_gu + (size_t)(l.sh_inter ? 32 : l.sff) * wp, l.sff, W, wp);
+        if (l.sh_inter)
+            for (const char* nm : {"mlp.shared.gate", "mlp.shared.up"}) { TensorDest& d = m->tensors[lp + nm]; d.group = 32; d.group_stride = 64; }
+        want_matrix(m, lp + "mlp.shared.down", l.w_sh_down, W, l.sff, l.sff_p);
+        m->g_cols = std::max(m->g_cols, 2 * l.sff);
+        m->kout_p_max = std::max(m->kout_p_max, l.sff_p);
+    }
+#undef TRY
+#undef REQ
     return GTB_OK;
 }
 
@@ -1254,7 +1525,7 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
         if (c.tied_head) { TensorDest& d = m->tensors["embed"]; d.also = m->head; d.also_ld = wp; }     // the product wants padded rows: a copy of its own
         else want_matrix(m, "head", m->head, c.vocab, W, wp);
     }
-    REQ(c.final_norm >= 0 && c.final_norm <= 4);
+    REQ(c.final_norm >= 0 && c.final_norm <= 5);
     REQ(c.streams >= 0 && c.streams <= HC_MAX && c.logit_softcap >= 0.0f);
     TRY(dalloc_t(m, &m->final_gain, c.final_norm ? W : 1));
     if (c.final_norm) want_vector(m, "final.norm", m->final_gain, W, 0);
@@ -1288,6 +1559,11 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
     for (int i = 0; i < c.n_layers; i++) {
         LayerW& l = m->L[i];
         l.d = layers[i];
+        if (l.d.weights_of >= 0) {               // another run of an earlier layer: no tensors here (add_run names the layer it runs)
+            REQ(l.d.weights_of < i && m->L[l.d.weights_of].d.weights_of < 0 && c.loop_times == 0);
+            l.d.n_branches = 0; l.d.ff = 0;
+            continue;
+        }
         const bool post = l.d.style == GTB_BLOCK_POSTNORM, pre = l.d.style == GTB_BLOCK_PRENORM, sw = l.d.style == GTB_BLOCK_SANDWICH;
         REQ(l.d.style == GTB_BLOCK_PARALLEL || post || pre || sw);
         REQ(pre == m->prenorm);                  // the copies of the stream belong to the whole model: pre-norm layers do not mix with the other styles
@@ -1295,9 +1571,11 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
         REQ(!(pre || sw) || (c.loop_times == 0 && c.taps == 0));
         REQ(l.d.n_branches >= 1 && l.d.n_branches <= (post || pre ? 1 : 2));
         if (l.d.n_branches == 2) for (const gtb_seq_branch& d : l.d.branch) REQ(d.kind != GTB_MIX_LATENT_ATTN && d.out_bias == 0);
+        REQ(l.d.join_norm == 0 || (l.d.join_norm == 1 && sw && l.d.n_branches == 2));
+        REQ(l.d.route_kind == GTB_ROUTE_LOGISTIC || (l.d.route_kind == GTB_ROUTE_SOFTMAX && l.d.ff_kind == GTB_FF_GATED_EXPERTS && l.d.shared_ff == 0));
         REQ(l.d.ff >= 0);
         if (sw) REQ((l.d.norm_kind == GTB_NORM_RMS || l.d.norm_kind == GTB_NORM_LAYER || l.d.norm_kind == GTB_NORM_LAYER_NB) &&
-                    (l.d.ff == 0 || l.d.ff_kind == GTB_FF_SWIGLU || l.d.ff_kind == GTB_FF_GROUP_EXPERTS || l.d.ff_kind == GTB_FF_GELU));
+                    (l.d.ff == 0 || l.d.ff_kind == GTB_FF_SWIGLU || l.d.ff_kind == GTB_FF_GROUP_EXPERTS || l.d.ff_kind == GTB_FF_GELU || l.d.ff_kind == GTB_FF_GATED_EXPERTS));
         else if (pre) REQ((l.d.norm_kind == GTB_NORM_RMS || l.d.norm_kind == GTB_NORM_DYT) && (l.d.ff == 0 || l.d.ff_kind == GTB_FF_GEGLU || l.d.ff_kind == GTB_FF_GATED_EXPERTS));
         else REQ(post ? (l.d.ff == 0 || l.d.ff_kind == GTB_FF_POLYNORM || l.d.ff_kind == GTB_FF_EXPERTS) : l.d.ff_kind == GTB_FF_GEGLU);
         l.ff = l.d.ff;
@@ -1308,11 +1586,47 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
             b.d = l.d.branch[bi];
             gtb_seq_branch& d = b.d;
             REQ(pre ? d.kind == GTB_MIX_LATENT_ATTN : post ? (d.kind == GTB_MIX_MINGRU || d.kind == GTB_MIX_SOFTMAX_ATTN) :
-                sw ? (d.kind == GTB_MIX_SOFTMAX_ATTN || d.kind == GTB_MIX_RETENTION || d.kind == GTB_MIX_LATENT_ATTN) : (d.kind == GTB_MIX_SIGMOID_ATTN || d.kind == GTB_MIX_RETENTION));
+                sw ? (d.kind == GTB_MIX_SOFTMAX_ATTN || d.kind == GTB_MIX_RETENTION || d.kind == GTB_MIX_LATENT_ATTN || rec_kind(d.kind) || d.kind == GTB_MIX_SSM) : (d.kind == GTB_MIX_SIGMOID_ATTN || d.kind == GTB_MIX_RETENTION));
             REQ(d.rot_scaling == GTB_ROT_SCALE_WAVES || d.rot_scaling == GTB_ROT_SCALE_YARN);
             if (d.rot_factor > 0.0f) REQ(d.rot_original > 0.0f && d.rot_base > 1.0f && d.rot_low > 0.0f && d.rot_high > 0.0f);
-            if (!sw || d.kind != GTB_MIX_SOFTMAX_ATTN) REQ(d.conv == 0 && d.v_from_k == 0 && d.keep_first == 0 && d.slopes == 0);
-            REQ(d.out_bias == 0 || (sw && d.kind != GTB_MIX_RETENTION));
+            if (!sw || d.kind != GTB_MIX_SOFTMAX_ATTN) REQ((d.conv == 0 || d.kind == GTB_MIX_DELTA || d.kind == GTB_MIX_SSM) && d.v_from_k == 0 && d.keep_first == 0 && d.slopes == 0);
+            REQ(d.out_bias == 0 || (sw && (d.kind == GTB_MIX_SOFTMAX_ATTN || d.kind == GTB_MIX_LATENT_ATTN)));
+            if (l.d.join_norm) ko = pad64(ko);       // an out projection of its own starts on a k-block
+            if (rec_kind(d.kind)) {
+                if (d.kind == GTB_MIX_MLSTM) d.kv_heads = d.heads;
+                REQ(d.heads > 0 && d.kv_heads > 0 && d.heads % d.kv_heads == 0 && d.dim > 0 && d.dim <= 1024 && d.vdim > 0 && d.scale > 0.0f);
+                REQ(d.kind == GTB_MIX_MLSTM ? (d.gate_cap > 0.0f && d.conv == 0) : (d.conv >= 1 && d.conv <= 64));
+                b.kq = b.kk = d.kv_heads * d.dim; b.kv = d.heads * d.vdim;
+                b.q_off = n1; b.k_off = b.q_off + b.kq; b.v_off = b.k_off + b.kk; b.g_off = b.v_off + b.kv; b.i_off = b.g_off + b.kv; b.f_off = b.i_off + d.heads;
+                n1 = b.f_off + d.heads;
+                b.a_off = ko; ko += b.kv; b.ko_p = pad64(b.kv);
+                m->rec_heads_max = std::max(m->rec_heads_max, d.heads);
+                m->ro_max = std::max(m->ro_max, d.heads * rec_vx(d));
+                if (d.kind == GTB_MIX_DELTA) m->conv_q_max = std::max(m->conv_q_max, b.kq + b.kk + b.kv);
+                if (const int C = rec_chunk(d)) {
+                    const RecBranch ra = rec_args(m, b);
+                    m->rec_qk_max = std::max(m->rec_qk_max, (size_t)m->max_rows * ra.kv_heads * ra.dp);
+                    m->rec_v_max = std::max(m->rec_v_max, (size_t)m->max_rows * ra.heads * ra.vp);
+                    if (d.kind == GTB_MIX_DELTA) m->rec_w_max = std::max(m->rec_w_max, (size_t)m->max_rows * ra.heads * ra.dp);
+                    m->rec_s_max = std::max(m->rec_s_max, (size_t)(m->max_rows / C + c.n_slots + 1) * ra.heads * 2 * ra.dp * ra.vp);
+                }
+                continue;
+            }
+            if (d.kind == GTB_MIX_SSM) {
+                REQ(d.inner > 0 && d.state > 0 && d.state <= 256 && d.dt_rank > 0 && d.conv >= 1 && d.conv <= 64);
+                d.heads = d.kv_heads = 1;
+                b.q_off = n1; n1 += 2 * d.inner;                 // x | z
+                b.a_off = ko; ko += d.inner; b.ko_p = pad64(d.inner);
+                b.ld_x = pad64(d.inner); b.dt_p = pad64(d.dt_rank); b.ld_bc = pad64(d.dt_rank + 2 * d.state);
+                m->conv_q_max = std::max(m->conv_q_max, d.inner);
+                m->ssm_inner_max = std::max(m->ssm_inner_max, d.inner);
+                m->ssm_bc_max = std::max(m->ssm_bc_max, b.ld_bc);
+                m->ssm_x_max = std::max(m->ssm_x_max, b.ld_x);
+                m->ssm_dt_max = std::max(m->ssm_dt_max, b.dt_p);
+                continue;
+            }
+            REQ(!l.d.join_norm || d.kind == GTB_MIX_SOFTMAX_ATTN);
+            b.ko_p = pad64(d.heads * d.vdim);
             if (d.kind == GTB_MIX_LATENT_ATTN) {
                 REQ(d.heads > 0 && d.dim > 0 && d.rope_dim >= 0 && d.vdim > 0 && d.kv_rank > 0 && d.q_rank >= 0 && d.window >= 0);
                 REQ(d.kv_rank <= 512 && d.kv_rank + d.rope_dim <= 1024);        // the absorbed form runs on the row kernels of softmax attention
@@ -1427,6 +1741,53 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
                 want_matrix(m, bp + "o", l.w_out + b.a_off, W, d.dim, l.kout_p);
                 continue;
             }
+            if (l.d.join_norm) { TRY(dalloc_t(m, &b.d_join, W)); want_vector(m, bp + "out", b.d_join, W, 0); m->join = true; }
+            if (rec_kind(d.kind)) {
+                const bool ml = d.kind == GTB_MIX_MLSTM;
+                want_matrix(m, bp + "q", l.w_mix + (size_t)b.q_off * wp, b.kq, W, wp);
+                want_matrix(m, bp + "k", l.w_mix + (size_t)b.k_off * wp, b.kk, W, wp);
+                want_matrix(m, bp + "v", l.w_mix + (size_t)b.v_off * wp, b.kv, W, wp);
+                want_matrix(m, bp + "g", l.w_mix + (size_t)b.g_off * wp, b.kv, W, wp);
+                want_matrix(m, bp + (ml ? "i" : "a"), l.w_mix + (size_t)b.i_off * wp, d.heads, W, wp);
+                want_matrix(m, bp + (ml ? "f" : "b"), l.w_mix + (size_t)b.f_off * wp, d.heads, W, wp);
+                if (ml) {
+                    if (!l.d_bias) TRY(dalloc_t(m, &l.d_bias, n1));
+                    want_vector(m, bp + "i.b", l.d_bias + b.i_off, d.heads, 0);
+                    want_vector(m, bp + "f.b", l.d_bias + b.f_off, d.heads, 0);
+                } else {
+                    TRY(dalloc_t(m, &b.d_Alog, d.heads));
+                    TRY(dalloc_t(m, &b.d_dtb, d.heads));
+                    want_vector(m, bp + "A_log", b.d_Alog, d.heads, 0);
+                    want_vector(m, bp + "dt_bias", b.d_dtb, d.heads, 0);
+                    TRY(dalloc_t(m, &b.d_conv, (size_t)(b.kq + b.kk + b.kv) * d.conv));      // one table: q, k, v channels
+                    want_vector(m, bp + "q.conv", b.d_conv, b.kq, d.conv);
+                    want_vector(m, bp + "k.conv", b.d_conv + (size_t)b.kq * d.conv, b.kk, d.conv);
+                    want_vector(m, bp + "v.conv", b.d_conv + (size_t)(b.kq + b.kk) * d.conv, b.kv, d.conv);
+                }
+                TRY(dalloc_t(m, &b.d_onorm, ml ? b.kv : d.vdim));
+                want_vector(m, bp + "norm", b.d_onorm, ml ? b.kv : d.vdim, 0);
+                want_matrix(m, bp + "o", l.w_out + b.a_off, W, b.kv, l.kout_p);
+                continue;
+            }
+            if (d.kind == GTB_MIX_SSM) {
+                want_matrix(m, bp + "in", l.w_mix + (size_t)b.q_off * wp, 2 * d.inner, W, wp);
+                TRY(dalloc_t(m, &b.d_conv, (size_t)d.inner * d.conv));
+                want_vector(m, bp + "conv", b.d_conv, d.inner, d.conv);
+                TRY(dalloc_t(m, &b.d_cbias, d.inner));
+                want_vector(m, bp + "conv.b", b.d_cbias, d.inner, 0);
+                TRY(dalloc_t(m, &b.w_x, (size_t)(d.dt_rank + 2 * d.state) * b.ld_x));
+                want_matrix(m, bp + "x", b.w_x, d.dt_rank + 2 * d.state, d.inner, b.ld_x);
+                TRY(dalloc_t(m, &b.w_dt, (size_t)d.inner * b.dt_p));
+                want_matrix(m, bp + "dt", b.w_dt, d.inner, d.dt_rank, b.dt_p);
+                TRY(dalloc_t(m, &b.d_dtb, d.inner));
+                want_vector(m, bp + "dt.b", b.d_dtb, d.inner, 0);
+                TRY(dalloc_t(m, &b.d_Alog, (size_t)d.inner * d.state));
+                want_vector(m, bp + "A_log", b.d_Alog, d.inner, d.state);
+                TRY(dalloc_t(m, &b.d_D, d.inner));
+                want_vector(m, bp + "D", b.d_D, d.inner, 0);
+                want_matrix(m, bp + "o", l.w_out + b.a_off, W, d.inner, l.kout_p);
+                continue;
+            }
             if (d.kind == GTB_MIX_LATENT_ATTN) {
                 const int hd = d.dim + d.rope_dim;
                 if (d.q_rank > 0) {
@@ -1529,6 +1890,8 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
                     want_matrix(m, lp + "mlp.down", l.w_down, W, l.ff, l.kfp);
                     m->g_cols = std::max(m->g_cols, l.ff);
                     m->kout_p_max = std::max(m->kout_p_max, l.kfp);
+                } else if (l.d.ff_kind == GTB_FF_GATED_EXPERTS) {
+                    TRY(want_gated_experts(m, l, lp));
                 } else {
                     const int E = l.d.experts, G = std::max(1, l.d.route_groups), keep = l.d.route_keep > 0 ? l.d.route_keep : G;
                     REQ(E > 0 && E <= 4096 && l.d.identity == 0 && l.d.top > 0 && l.d.shared_ff >= 0 && E % G == 0 && keep <= G && l.d.top <= keep * (E / G));
@@ -1593,41 +1956,7 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
                     m->g_cols = std::max(m->g_cols, 2 * l.ff);
                     m->kout_p_max = std::max(m->kout_p_max, l.kfp);
                 } else {
-                    const int E = l.d.experts;
-                    REQ(E > 0 && E <= 4096 && l.d.identity == 0 && l.d.top > 0 && l.d.top <= E && l.d.top <= 64 && l.d.shared_ff >= 0);
-                    l.sff = l.d.shared_ff;
-                    l.n_out = E + (l.sff > 0 ? 1 : 0);
-                    TRY(dalloc_t(m, &l.w_router, (size_t)l.n_out * wp));
-                    want_matrix(m, lp + "mlp.router", l.w_router, E, W, wp);
-                    if (l.sff > 0) want_matrix(m, lp + "mlp.shared.sg", l.w_router + (size_t)E * wp, 1, W, wp);
-                    TRY(dalloc_t(m, &l.w_up, (size_t)E * 2 * l.ff * wp));
-                    TRY(dalloc_t(m, &l.w_down, (size_t)E * W * l.kfp));
-                    l.e_inter = l.ff % 32 == 0;
-                    for (int e = 0; e < E; e++) {
-                        const std::string ep = lp + "mlp.e" + std::to_string(e) + ".";
-                        bf16* base = l.w_up + (size_t)e * 2 * l.ff * wp;
-                        want_matrix(m, ep + "gate", base, l.ff, W, wp);
-                        want_matrix(m, ep + "up", base + (size_t)(l.e_inter ? 32 : l.ff) * wp, l.ff, W, wp);
-                        if (l.e_inter)
-                            for (const char* nm : {"gate", "up"}) { TensorDest& d = m->tensors[ep + nm]; d.group = 32; d.group_stride = 64; }
-                        want_matrix(m, ep + "down", l.w_down + (size_t)e * W * l.kfp, W, l.ff, l.kfp);
-                    }
-                    m->n_out_max = std::max(m->n_out_max, l.n_out);
-                    m->top_max = std::max(m->top_max, l.d.top);
-                    m->e_max = std::max(m->e_max, E);
-                    if (l.sff > 0) {
-                        l.sff_p = pad64(l.sff);
-                        l.sh_inter = l.sff % 32 == 0;
-                        TRY(dalloc_t(m, &l.w_sh_gu, (size_t)2 * l.sff * wp));
-                        TRY(dalloc_t(m, &l.w_sh_down, (size_t)W * l.sff_p));
-                        want_matrix(m, lp + "mlp.shared.gate", l.w_sh_gu, l.sff, W, wp);
-                        want_matrix(m, lp + "mlp.shared.up", l.w_sh_gu + (size_t)(l.sh_inter ? 32 : l.sff) * wp, l.sff, W, wp);
-                        if (l.sh_inter)
-                            for (const char* nm : {"mlp.shared.gate", "mlp.shared.up"}) { TensorDest& d = m->tensors[lp + nm]; d.group = 32; d.group_stride = 64; }
-                        want_matrix(m, lp + "mlp.shared.down", l.w_sh_down, W, l.sff, l.sff_p);
-                        m->g_cols = std::max(m->g_cols, 2 * l.sff);
-                        m->kout_p_max = std::max(m->kout_p_max, l.sff_p);
-                    }
+                    TRY(want_gated_experts(m, l, lp));
                 }
             }
         } else if (post) {
@@ -1702,7 +2031,7 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
             for (int i = c.loop_start; i < c.loop_stop; i++) add_run(i, p, i == c.loop_start);
         for (int i = c.loop_stop; i < c.n_layers; i++) add_run(i, -1, false);
     } else {
-        for (int i = 0; i < c.n_layers; i++) add_run(i, -1, false);
+        for (int i = 0; i < c.n_layers; i++) add_run(m->L[i].d.weights_of >= 0 ? m->L[i].d.weights_of : i, -1, false);
     }
     for (const Run& r : m->runs) REQ(!(r.enters_pass && m->L[r.layer].d.style == GTB_BLOCK_POSTNORM));      // a loop pass opens with a parallel block
     // state of every run, for every slot
@@ -1746,6 +2075,13 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
                 const size_t sb = state_floats(d) * sizeof(float);
                 TRY(dalloc(m, (void**)&r.state[bi], sb * c.n_slots));
                 per_slot += sb;
+                if (d.kind == GTB_MIX_MLSTM) { TRY(dalloc_t(m, &r.mstate[bi], (size_t)c.n_slots * d.heads)); per_slot += d.heads * sizeof(float); }
+                if ((d.kind == GTB_MIX_DELTA || d.kind == GTB_MIX_SSM) && d.conv > 1) {
+                    REQ(!r.ctail);
+                    r.ctail_n = (d.conv - 1) * (d.kind == GTB_MIX_SSM ? d.inner : l.br[bi].kq + l.br[bi].kk + l.br[bi].kv);
+                    TRY(dalloc_t(m, &r.ctail, (size_t)c.n_slots * r.ctail_n));
+                    per_slot += r.ctail_n * sizeof(float);
+                }
             }
         }
         if (c.taps > 1) {
@@ -1777,8 +2113,10 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
     {
         size_t hv = 0;
         for (const LayerW& l : m->L)
-            if (l.br[0].d.kind == GTB_MIX_SOFTMAX_ATTN) hv = std::max(hv, (size_t)l.br[0].d.heads * std::max(1, l.br[0].d.maps) * (l.br[0].d.vdim + 2));
-            else if (l.br[0].d.kind == GTB_MIX_LATENT_ATTN) hv = std::max(hv, (size_t)l.br[0].d.heads * (l.br[0].d.kv_rank + 2));
+            if (l.br[0].d.kind == GTB_MIX_SOFTMAX_ATTN || l.br[1].d.kind == GTB_MIX_SOFTMAX_ATTN) {
+                for (const BranchW& b : l.br)
+                    if (b.d.kind == GTB_MIX_SOFTMAX_ATTN) hv = std::max(hv, (size_t)b.d.heads * std::max(1, b.d.maps) * (b.d.vdim + 2));
+            } else if (l.br[0].d.kind == GTB_MIX_LATENT_ATTN) hv = std::max(hv, (size_t)l.br[0].d.heads * (l.br[0].d.kv_rank + 2));
         if (hv > 0 && c.max_ctx > 128) TRY(dalloc_t(m, &m->sattn_part, 32 * SPLIT_MAX_ROWS * hv));
     }
     if (m->n_out_max > 0) {
@@ -1807,8 +2145,27 @@ int gtb_seq_create(gtb_seq_t* out, const gtb_seq_config* cfg, const gtb_seq_laye
     if (m->conv_q_max > 0) TRY(dalloc_t(m, &m->convQ, R * m->conv_q_max));
     if (m->prenorm) {
         TRY(dalloc_t(m, &m->xs, (size_t)m->ns * R * W));
+    }
+    if (m->prenorm || m->sandwich) {         // a second share of a sublayer's output: shared expert, second branch
         TRY(dalloc_t(m, &m->Y2, R * W));
         TRY(dalloc_t(m, &m->shw, R));
+    }
+    if (m->rec_heads_max > 0) {
+        TRY(dalloc_t(m, &m->recG, R * m->rec_heads_max));
+        if (c.mode == GTB_SEQ_BF16 && m->rec_qk_max > 0) {
+            TRY(dalloc_t(m, &m->recB, R * m->rec_heads_max));
+            TRY(dalloc_t(m, &m->recQ, 2 * m->rec_qk_max));
+            TRY(dalloc_t(m, &m->recK, 2 * m->rec_qk_max));
+            TRY(dalloc_t(m, &m->recV, 2 * m->rec_v_max));
+            TRY(dalloc_t(m, &m->recW, 2 * m->rec_w_max));
+            TRY(dalloc_t(m, &m->recS, m->rec_s_max));
+        }
+    }
+    if (m->ssm_inner_max > 0) {
+        TRY(dalloc_t(m, &m->ssmBC, R * m->ssm_bc_max));
+        TRY(dalloc_t(m, &m->ssmDT, R * m->ssm_inner_max));
+        TRY(dalloc(m, &m->opX, R * m->ssm_x_max * es));
+        TRY(dalloc(m, &m->opDT, R * m->ssm_dt_max * es));
     }
     if (m->lat_q_max > 0) {
         TRY(dalloc_t(m, &m->latQ, R * std::max(m->lat_q_max, 1)));
@@ -1914,6 +2271,7 @@ int gtb_seq_slot_reset(gtb_seq_t m, int slot) {
             if (r.state[bi]) {
                 const size_t sb = state_floats(l.br[bi].d) * sizeof(float);
                 GTB_CUDA(cudaMemsetAsync((char*)r.state[bi] + sb * slot, 0, sb, st));
+                if (r.mstate[bi]) GTB_CUDA(cudaMemsetAsync(r.mstate[bi] + (size_t)l.br[bi].d.heads * slot, 0, l.br[bi].d.heads * sizeof(float), st));
             }
         if (r.ctail) GTB_CUDA(cudaMemsetAsync(r.ctail + (size_t)r.ctail_n * slot, 0, r.ctail_n * sizeof(float), st));
         if (r.tail) {

@@ -5,8 +5,10 @@
 //   * one RMS norm over a whole query / key projection (its scale per row), for softmax attention with qk_norm 3
 //   * differential attention: the combination of a head's two score maps, its unit-RMS norm and gate
 //   * retention with SiLU-activated inputs, an RMS norm over the concatenated heads and a logistic gate
-//   * a sigmoid router whose choice is limited to the best groups of experts
-//   * a short causal convolution right behind the query and key projections, with the cache append behind it
+//   * a sigmoid router whose choice is limited to the best groups of experts, and a router that weights the largest outputs with their own softmax
+//   * two branches with out projections and norms of their own, joined in the residual update
+//   * a short causal convolution right behind the query and key projections, with the cache append behind it (recurrent mixers: with a bias, silu and
+//     an operand copy)
 //   * the erf form of GELU as the activation of an ungated feed-forward
 // The attention and retention kernels themselves are those of gtb_seq_mixers*.cuh and gtb_seq_kernels.cuh.
 //
@@ -132,8 +134,42 @@ __global__ void __launch_bounds__(32) k_moe_route_grouped(const float* __restric
     route_grouped_row(Z + (size_t)r * ldz, n_exp, n_groups, keep, top, scale, n_always, sel_idx + (size_t)r * tt, sel_w + (size_t)r * tt, rsm, rsm + n_exp,
                       rsm + 2 * n_exp, threadIdx.x);
 }
+// One warp routes one row from its router outputs z [n_exp]: the `top` largest are chosen (ties to the lower index), their weights are the softmax
+// over the chosen outputs alone.  ch: n_exp floats of shared memory.
+__device__ __forceinline__ void route_top_softmax_row(const float* __restrict__ z, int n_exp, int top, int* __restrict__ sel_idx, float* __restrict__ sel_w, float* ch, int lane) {
+    for (int i = lane; i < n_exp; i += 32) ch[i] = z[i];
+    __syncwarp();
+    float first = 0.0f, sum = 0.0f, e0 = 0.0f, e1 = 0.0f;        // lane k % 32 keeps exp(z_k - z_0) of choice k (at most 64 choices)
+    for (int k = 0; k < top; k++) {
+        float best = -INFINITY;
+        int arg = 0x7fffffff;
+        for (int i = lane; i < n_exp; i += 32) { const float v = ch[i]; if (v > best) { best = v; arg = i; } }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, arg, o);
+            if (ov > best || (ov == best && oi < arg)) { best = ov; arg = oi; }
+        }
+        if (k == 0) first = best;
+        float e = expf(best - first);
+        if (arg == 0x7fffffff) { arg = 0; e = 0.0f; }            // every remaining output is -inf or NaN
+        sum += e;
+        if (lane == (k & 31)) { if (k < 32) e0 = e; else e1 = e; }
+        if (lane == 0) { sel_idx[k] = arg; ch[arg] = -INFINITY; }
+        __syncwarp();
+    }
+    const float inv = 1.0f / sum;
+    if (lane < top) sel_w[lane] = e0 * inv;
+    if (lane + 32 < top) sel_w[lane + 32] = e1 * inv;
+}
+__global__ void __launch_bounds__(32) k_moe_route_softmax(const float* __restrict__ Z, int ldz, int n_exp, int top, int* __restrict__ sel_idx, float* __restrict__ sel_w) {
+    extern __shared__ float rsm[];
+    const int r = blockIdx.x;
+    route_top_softmax_row(Z + (size_t)r * ldz, n_exp, top, sel_idx + (size_t)r * top, sel_w + (size_t)r * top, rsm, threadIdx.x);
+}
 // The router of the NEXT sublayer inside the residual update (few rows): what k_sandwich_add appends when it is given a router
 struct GroupRouteNext {
+    int kind;                  // 0: group-limited logistic; 1: softmax over the chosen outputs (groups, scale and n_always unused)
     const bf16* w;             // [n_exp][ldw] router matrix, or null: no routing here
     int ldw, n_exp, n_groups, keep, top, n_always;
     float scale;
@@ -165,7 +201,8 @@ __device__ __forceinline__ void sandwich_route(const GroupRouteNext& rn, float* 
     }
     __syncthreads();
     const int tt = rn.top + rn.n_always;
-    if (wid == 0)
+    if (wid == 0 && rn.kind == 1) route_top_softmax_row(sl, rn.n_exp, rn.top, rn.sel_idx + (size_t)r * rn.top, rn.sel_w + (size_t)r * rn.top, sl + rn.n_exp, lane);
+    else if (wid == 0)
         route_grouped_row(sl, rn.n_exp, rn.n_groups, rn.keep, rn.top, rn.scale, rn.n_always, rn.sel_idx + (size_t)r * tt, rn.sel_w + (size_t)r * tt, sl + rn.n_exp,
                           sl + 2 * rn.n_exp, sl + 3 * rn.n_exp, lane);
 }
@@ -192,13 +229,15 @@ __global__ void __launch_bounds__(256) k_embed_norm(PassTables t, const bf16* __
 // stay in registers between the passes (16-byte accesses); wider or unaligned rows walk the row again.  With a router (rn.w; few rows) the
 // kernel also forms the next sublayer's router logits from the operand row it has just written and picks the experts; dynamic shared
 // memory: width + 3 n_exp + n_groups floats.
+// JOIN: Y and Y2 are two branches, y = scale (Y / rms(Y) w1 + Y2 / rms(Y2) w2), each norm over the row with its own weight.
 // SW_KEEP: float4 groups a thread keeps per array (1, 2 or 4: rows up to 1024, 2048, 4096 wide); fewer kept values, fewer registers, more rows
 // in flight per SM -- the kernel is bound by the latency of a row's load / reduce / store chain, not by bandwidth.
-template <typename OT, int SW_KEEP>
-__global__ void __launch_bounds__(256, SW_KEEP == 4 ? 4 : SW_KEEP == 2 ? 6 : 8) k_sandwich_add(const float* __restrict__ Y, const float* __restrict__ Y2, const float* __restrict__ Yg,
+struct JoinArgs { const float *w1, *w2; float scale, eps; };
+template <typename OT, int SW_KEEP, bool JOIN = false>
+__global__ void __launch_bounds__(256, JOIN ? (SW_KEEP == 4 ? 2 : 4) : SW_KEEP == 4 ? 4 : SW_KEEP == 2 ? 6 : 8) k_sandwich_add(const float* __restrict__ Y, const float* __restrict__ Y2, const float* __restrict__ Yg,
                                                       const int* __restrict__ pair_dst, int top, int width, NormArgs post, float* __restrict__ x,
-                                                      NormArgs next, OT* __restrict__ op, int ld_op, GroupRouteNext rn) {
-    __shared__ float red[128];           // four reductions, each with 32 floats of its own (the walking path uses the first 33)
+                                                      NormArgs next, OT* __restrict__ op, int ld_op, GroupRouteNext rn, JoinArgs jn) {
+    __shared__ float red[JOIN ? 192 : 128];           // four reductions (two more to join branches), each with 32 floats of its own (the walking path uses the first 33)
     __shared__ int sdst[PN_MAX_TOP];
     extern __shared__ float srt[];
     const int r = blockIdx.x;
@@ -214,8 +253,8 @@ __global__ void __launch_bounds__(256, SW_KEEP == 4 ? 4 : SW_KEEP == 2 ? 6 : 8) 
             if (c < width) {
                 float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
                 if (Y) y = *reinterpret_cast<const float4*>(Y + (size_t)r * width + c);
-                if (Y2) { const float4 t4 = *reinterpret_cast<const float4*>(Y2 + (size_t)r * width + c); y.x += t4.x; y.y += t4.y; y.z += t4.z; y.w += t4.w; }
-                if (Yg)
+                if (!JOIN && Y2) { const float4 t4 = *reinterpret_cast<const float4*>(Y2 + (size_t)r * width + c); y.x += t4.x; y.y += t4.y; y.z += t4.z; y.w += t4.w; }
+                if (!JOIN && Yg)
                     for (int k = 0; k < top; k++)
                         if (sdst[k] >= 0) { const float4 t4 = *reinterpret_cast<const float4*>(Yg + (size_t)sdst[k] * width + c); y.x += t4.x; y.y += t4.y; y.z += t4.z; y.w += t4.w; }
                 const float4 xv = *reinterpret_cast<const float4*>(xr + c);
@@ -224,6 +263,26 @@ __global__ void __launch_bounds__(256, SW_KEEP == 4 ? 4 : SW_KEEP == 2 ? 6 : 8) 
             }
         }
         float mean, rstd;
+        if constexpr (JOIN) {
+            float v2[4 * SW_KEEP], r1, r2;
+#pragma unroll
+            for (int i = 0; i < SW_KEEP; i++) {
+                const int c = (threadIdx.x + i * blockDim.x) * 4;
+                if (c < width) { const float4 t4 = *reinterpret_cast<const float4*>(Y2 + (size_t)r * width + c); v2[4 * i] = t4.x; v2[4 * i + 1] = t4.y; v2[4 * i + 2] = t4.z; v2[4 * i + 3] = t4.w; }
+            }
+            sw_stats<SW_KEEP>(vy, width, 0, jn.eps, red + 128 - 32, mean, r1);       // (RMS uses the second 32 floats it is given)
+            sw_stats<SW_KEEP>(v2, width, 0, jn.eps, red + 160 - 32, mean, r2);
+            r1 *= jn.scale; r2 *= jn.scale;
+#pragma unroll
+            for (int i = 0; i < SW_KEEP; i++) {
+                const int c = (threadIdx.x + i * blockDim.x) * 4;
+                if (c < width) {
+                    const float4 a4 = *reinterpret_cast<const float4*>(jn.w1 + c), b4 = *reinterpret_cast<const float4*>(jn.w2 + c);
+                    vy[4 * i] = vy[4 * i] * r1 * a4.x + v2[4 * i] * r2 * b4.x; vy[4 * i + 1] = vy[4 * i + 1] * r1 * a4.y + v2[4 * i + 1] * r2 * b4.y;
+                    vy[4 * i + 2] = vy[4 * i + 2] * r1 * a4.z + v2[4 * i + 2] * r2 * b4.z; vy[4 * i + 3] = vy[4 * i + 3] * r1 * a4.w + v2[4 * i + 3] * r2 * b4.w;
+                }
+            }
+        }
         sw_stats<SW_KEEP>(vy, width, cp, post.eps, red, mean, rstd);
 #pragma unroll
         for (int i = 0; i < SW_KEEP; i++) {
@@ -254,7 +313,14 @@ __global__ void __launch_bounds__(256, SW_KEEP == 4 ? 4 : SW_KEEP == 2 ? 6 : 8) 
         if (rn.w) sandwich_route(rn, srt, width, r);
         return;
     }
+    float j1 = 0.0f, j2 = 0.0f;
+    if (JOIN) {
+        for (int c = threadIdx.x; c < width; c += blockDim.x) { const float a = Y[(size_t)r * width + c], q = Y2[(size_t)r * width + c]; j1 += a * a; j2 += q * q; }
+        j1 = jn.scale / sqrtf(block_sum(j1, red) / (float)width + jn.eps);
+        j2 = jn.scale / sqrtf(block_sum(j2, red) / (float)width + jn.eps);
+    }
     auto sub = [&](int c) {
+        if (JOIN) return Y[(size_t)r * width + c] * j1 * jn.w1[c] + Y2[(size_t)r * width + c] * j2 * jn.w2[c];
         float a = Y ? Y[(size_t)r * width + c] : 0.0f;
         if (Y2) a += Y2[(size_t)r * width + c];
         if (Yg)
@@ -364,6 +430,10 @@ struct ConvArgs {
     int taps;
     const float* w;              // [nq + nk][taps]
     int max_ctx, k_ld, v_ld;     // cache rows
+    const float* bias;           // [nq + nk] added behind the convolution, or null
+    int silu;                    // 1: silu on the result
+    void* op;                    // the convolved "queries" once more as a product operand [R][ld_op], or null
+    int ld_op;
 };
 // y_t = sum_j w[c][j] u_(t - taps + 1 + j) of every query and key channel of P; queries -> Q [R][nq] (fp32), keys -> the slot's key cache.
 // Rows before the segment come from the slot's history `tail` [n_slots][taps - 1][nq + nk] (zeros after a reset = zeros before the
@@ -444,6 +514,15 @@ __global__ void __launch_bounds__(128) k_qk_conv(PassTables t, ConvArgs b, const
                     y[i] = fmaf(b.w[(size_t)(c + i) * b.taps + j], src >= row0 ? p[(size_t)src * ldp + i] : tl[(size_t)(src - row0 + b.taps - 1) * nc + i], y[i]);
             }
         }
+        if (b.bias) {
+#pragma unroll
+            for (int i = 0; i < V; i++) y[i] += b.bias[c + i];
+        }
+        if (b.silu) {
+#pragma unroll
+            for (int i = 0; i < V; i++) y[i] = silu_(y[i]);
+        }
+        if (b.op && c < b.nq) cv_store(reinterpret_cast<OT*>(b.op) + (size_t)r * b.ld_op + c, y);
         if (c < b.nq) cv_store(Q + (size_t)r * b.nq + c, y);
         else cv_store(kc + ((size_t)slot * b.max_ctx + t.row_pos[r]) * b.k_ld + (c - b.nq), y);
     }

@@ -60,8 +60,13 @@ def _open_bisodra(path: Path, dtype: str, n_slots: int, max_ctx: int, **kw):
     return _open_described(bisodra, path, dtype, n_slots, max_ctx, **kw)
 
 
-FAMILIES = {"Bisodra": _open_bisodra, "Nanotar": _open_nanotar, "Reninex": _open_reninex, "Robopel": _open_robopel, "TinyLlama": _open_tinyllama, "Vulosun": _open_vulosun}
-STEPWISE = {"Bisodra", "Nanotar", "Reninex", "Robopel", "Vulosun"}          # families of the layer-list library: slots, portion-wise step function, scheduler
+def _open_siladra(path: Path, dtype: str, n_slots: int, max_ctx: int, **kw):
+    from . import siladra
+    return _open_described(siladra, path, dtype, n_slots, max_ctx, **kw)
+
+
+FAMILIES = {"Bisodra": _open_bisodra, "Nanotar": _open_nanotar, "Reninex": _open_reninex, "Robopel": _open_robopel, "Siladra": _open_siladra, "TinyLlama": _open_tinyllama, "Vulosun": _open_vulosun}
+STEPWISE = {"Bisodra", "Nanotar", "Reninex", "Robopel", "Siladra", "Vulosun"}          # families of the layer-list library: slots, portion-wise step function, scheduler
 
 
 def family_of(path) -> str:

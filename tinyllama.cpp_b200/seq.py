@@ -13,9 +13,11 @@ LIB_PATH = HERE / "libgten_b200_seq.so"
 
 BF16, F32 = 0, 1
 MIX_SIGMOID_ATTN, MIX_RETENTION, MIX_MINGRU, MIX_SOFTMAX_ATTN, MIX_LATENT_ATTN = 1, 2, 3, 4, 5
+MIX_MLSTM, MIX_DELTA, MIX_SSM = 6, 7, 8
 BLOCK_PARALLEL, BLOCK_POSTNORM, BLOCK_PRENORM, BLOCK_SANDWICH = 0, 1, 2, 3
 FF_GEGLU, FF_POLYNORM, FF_EXPERTS, FF_GATED_EXPERTS, FF_SWIGLU, FF_GROUP_EXPERTS, FF_GELU = 0, 1, 2, 3, 4, 5, 6
 NORM_RMS, NORM_DYT, NORM_LAYER, NORM_LAYER_NB = 0, 1, 2, 3
+ROUTE_LOGISTIC, ROUTE_SOFTMAX = 0, 1
 ROT_HALVES, ROT_INTERLEAVED = 0, 1
 ROT_SCALE_WAVES, ROT_SCALE_YARN = 0, 1
 MODE_BY_NAME = {"bfloat16": BF16, "bf16": BF16, "float32": F32, "fp32": F32}
@@ -33,13 +35,15 @@ class BranchC(C.Structure):
                 ("window", C.c_int), ("pool", C.c_int), ("sink", C.c_int), ("kv_from", C.c_int),
                 ("rope_dim", C.c_int), ("kv_rank", C.c_int), ("q_rank", C.c_int),
                 ("chunk", C.c_int), ("maps", C.c_int), ("diff", C.c_float), ("bias", C.c_int), ("act", C.c_int), ("rot_divide", C.c_float),
-                ("rot_scaling", C.c_int), ("conv", C.c_int), ("v_from_k", C.c_int), ("keep_first", C.c_int), ("slopes", C.c_int), ("out_bias", C.c_int)]
+                ("rot_scaling", C.c_int), ("conv", C.c_int), ("v_from_k", C.c_int), ("keep_first", C.c_int), ("slopes", C.c_int), ("out_bias", C.c_int),
+                ("gate_cap", C.c_float), ("inner", C.c_int), ("state", C.c_int), ("dt_rank", C.c_int)]
 
 
 class LayerC(C.Structure):
     _fields_ = [("n_branches", C.c_int), ("branch", BranchC * 2), ("ff", C.c_int), ("style", C.c_int), ("ff_kind", C.c_int),
                 ("experts", C.c_int), ("top", C.c_int), ("identity", C.c_int), ("norm_kind", C.c_int), ("shared_ff", C.c_int),
-                ("route_groups", C.c_int), ("route_keep", C.c_int), ("route_scale", C.c_float)]
+                ("route_groups", C.c_int), ("route_keep", C.c_int), ("route_scale", C.c_float),
+                ("route_kind", C.c_int), ("join_norm", C.c_int), ("weights_of", C.c_int)]
 
 
 class ConfigC(C.Structure):
@@ -130,7 +134,7 @@ class SeqModel:
 
     def __init__(self, desc: dict, mode: int, n_slots: int, max_ctx: int, max_rows: int = 0):
         """desc: the flat description a model family's config reader produces (see reninex.describe, robopel.describe, nanotar.describe,
-        vulosun.describe, bisodra.describe)."""
+        vulosun.describe, bisodra.describe, siladra.describe)."""
         self.desc, self.mode, self.n_slots, self.max_ctx = desc, mode, n_slots, max_ctx
         self.vocab, self.width = desc["vocab"], desc["width"]
         layers = (LayerC * len(desc["layers"]))()
@@ -142,10 +146,12 @@ class SeqModel:
             lc.experts, lc.top, lc.identity = l.get("experts", 0), l.get("top", 0), l.get("identity", 0)
             lc.norm_kind, lc.shared_ff = l.get("norm_kind", NORM_RMS), l.get("shared_ff", 0)
             lc.route_groups, lc.route_keep, lc.route_scale = l.get("route_groups", 0), l.get("route_keep", 0), l.get("route_scale", 1.0)
+            lc.route_kind, lc.join_norm, lc.weights_of = l.get("route_kind", ROUTE_LOGISTIC), int(l.get("join_norm", 0)), l.get("weights_of", -1)
             for bc, b in zip(lc.branch, l["branches"]):
                 bc.kind, bc.name = b["kind"], b["name"].encode()
-                bc.heads, bc.kv_heads, bc.dim, bc.vdim = b["heads"], b.get("kv_heads", b["heads"]), b["dim"], b["vdim"]
-                bc.scale, bc.qk_norm = b["scale"], int(b.get("qk_norm", 0))
+                bc.heads, bc.dim, bc.vdim = b.get("heads", 1), b.get("dim", 0), b.get("vdim", 0)
+                bc.kv_heads = b.get("kv_heads", bc.heads)
+                bc.scale, bc.qk_norm = b.get("scale", 1.0), int(b.get("qk_norm", 0))
                 bc.rot_dims, bc.rot_base = b.get("rot_dims", 0), b.get("rot_base", 10000.0)
                 bc.out_norm, bc.gated, bc.out_scale = int(b.get("out_norm", 0)), int(b.get("gated", 0)), b.get("out_scale", 1.0)
                 bc.rot_layout = b.get("rot_layout", ROT_HALVES)
@@ -157,6 +163,7 @@ class SeqModel:
                 bc.bias, bc.act, bc.rot_divide = int(b.get("bias", 0)), int(b.get("act", 0)), b.get("rot_divide", 0.0)
                 bc.rot_scaling, bc.conv, bc.v_from_k = b.get("rot_scaling", ROT_SCALE_WAVES), b.get("conv", 0), int(b.get("v_from_k", 0))
                 bc.keep_first, bc.slopes, bc.out_bias = b.get("keep_first", 0), int(b.get("slopes", 0)), int(b.get("out_bias", 0))
+                bc.gate_cap, bc.inner, bc.state, bc.dt_rank = b.get("gate_cap", 0.0), b.get("inner", 0), b.get("state", 0), b.get("dt_rank", 0)
                 if b.get("decay") is not None:
                     arr = (C.c_float * len(b["decay"]))(*b["decay"])
                     self._keep.append(arr)
