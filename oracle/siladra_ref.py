@@ -185,7 +185,7 @@ def route(z, top):
 
 
 def experts(h, T, c, book=None):
-    idx, w = route(h @ T["router"].T, c["router"]["top"])
+    idx, w = route(np.stack([h @ row for row in T["router"]], axis=-1), c["router"]["top"])
     out = np.zeros_like(h)
     for t in range(h.shape[0]):
         for e, wt in zip(idx[t], w[t]):

@@ -5,7 +5,8 @@ family beside Robopel (the closest existing model: softmax attention with a wind
 widths and layer count.  `bench.py --workload vulosun`: the Vulosun family beside Robopel (the closest existing model: sequential sublayers
 with norms on their outputs, softmax attention with a sink, a gate and a shared cache, squared-ReLU experts) at the same widths and layer
 count.  `bench.py --workload bisodra`: the Bisodra family beside Vulosun (the same layer style) and Nanotar (the same latent attention) at the
-same widths and layer count.  Timed with CUDA events on each library's own stream,
+same widths and layer count.  `bench.py --workload siladra`: the Siladra family beside Vulosun (the same layer style, a decayed recurrence beside
+softmax attention) and Nanotar (the same gated experts) at the same widths and layer count.  Timed with CUDA events on each library's own stream,
 after warm-up; the weights of one pass (hundreds of MB) are larger than L2, so every pass streams them from HBM."""
 from __future__ import annotations
 
@@ -620,6 +621,156 @@ def run_bisodra(args, root, clock_sampler) -> None:
                       "steps": iters, "warmup": warm, "ms_per_step": head["prefill"]["ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
                       "dtype": "bf16 operands, fp32 accumulation; fp32 stream, norms, convolution, scores", "data": "synthetic",
                       "config": {"workload": f"Bisodra {head['size']} x {head['layers']} layers, random weights: prefill of {T} tokens; decode at that context",
+                                 "l2": "weights of a pass exceed L2"},
+                      "detail": res, "gpu_launches": head["prefill_launches"], "clocks": clk.summary()}), flush=True)
+
+
+SILADRA_SIZES = {
+    # width; mLSTM heads x dim | vdim; delta-rule heads / q-k heads x dim | vdim, taps; parallel: attention heads / kv x dim, scan channels x states, step rank, taps;
+    # experts x ff (top)
+    "w2048": dict(width=2048, m_heads=8, m_dim=128, m_vdim=256, d_heads=16, d_kv=8, d_dim=128, d_vdim=128, conv=4, heads=16, kv=4, dim=64, inner=4096, state=16, dt_rank=128,
+                  experts=16, top=2, eff=1408),
+    "w1024": dict(width=1024, m_heads=4, m_dim=128, m_vdim=256, d_heads=8, d_kv=4, d_dim=128, d_vdim=128, conv=4, heads=8, kv=4, dim=64, inner=2048, state=16, dt_rank=64,
+                  experts=16, top=2, eff=704),
+}
+
+
+def siladra_config(name, vocab=32000):
+    """Four layers: mLSTM, parallel (attention | selective scan), gated delta rule, the first layer once more; all with experts."""
+    from . import siladra as SI
+    z = SILADRA_SIZES[name]
+    moe = lambda: SI.moe_mlp(ff=z["eff"], experts=z["experts"], top=z["top"])
+    layers = [SI.mlstm_layer(heads=z["m_heads"], dim=z["m_dim"], vdim=z["m_vdim"], gate_cap=15.0, mlp=moe()),
+              SI.parallel_layer(heads=z["heads"], kv_heads=z["kv"], dim=z["dim"], vdim=z["dim"], rot_dims=z["dim"], rot_base=100000.0, yarn=(4.0, 1024.0, 32.0, 1.0), inner=z["inner"],
+                                state=z["state"], dt_rank=z["dt_rank"], conv=z["conv"], mlp=moe()),
+              SI.delta_layer(heads=z["d_heads"], kv_heads=z["d_kv"], dim=z["d_dim"], vdim=z["d_vdim"], conv=z["conv"], mlp=moe())]
+    layers.append(SI.again(layers, 0))
+    return SI.make_config(vocab=vocab, width=z["width"], layers=layers, eps=1e-6, embed_scale=8.0)
+
+
+def siladra_counts(desc, T):
+    """(weights every token multiplies, FLOPs of the mixers' own arithmetic for a T-token prompt, bytes of weights a decode step of one
+    sequence reads) -- routed experts count `top` experts per token; recurrences count the state update and the read-out of every token (the delta
+    rule also what it reads before it writes); a layer that runs another one's tensors reads them again."""
+    from .seq import MIX_DELTA, MIX_MLSTM, MIX_SSM
+    W, params, mix = desc["width"], 0, 0.0
+    for l in desc["layers"]:
+        for b in l["branches"]:
+            if b["kind"] == MIX_SSM:
+                params += W * 3 * b["inner"] + b["inner"] * (2 * b["dt_rank"] + 2 * b["state"])
+                mix += 6.0 * b["inner"] * b["state"] * T
+                continue
+            H, G, D, V = b["heads"], b.get("kv_heads", b["heads"]), b["dim"], b["vdim"]
+            if b["kind"] == MIX_MLSTM:
+                params += W * (2 * H * D + 3 * H * V + 2 * H)
+                mix += 4.0 * H * D * (V + 1) * T
+            elif b["kind"] == MIX_DELTA:
+                params += W * (2 * G * D + 3 * H * V + 2 * H)
+                mix += 6.0 * H * D * V * T
+            else:
+                params += W * ((H + G) * D + (H + G) * V)
+                mix += 2.0 * H * (D + V) * T * (T + 1) / 2
+        if l["ff"]:
+            params += W * l["experts"] + l["top"] * 3 * W * l["ff"]
+    return params + desc["vocab"] * W, mix, 2 * (params + desc["vocab"] * W)
+
+
+def siladra_tensors(desc, rng):
+    """Cheap random weights of the right scale."""
+    from . import siladra as SI
+    tensors = {}
+    for k, shape in SI.tensor_shapes(desc).items():
+        n = int(np.prod(shape))
+        leaf = k.split(".")[-1]
+        if leaf.startswith("norm") or leaf in ("out", "D"):
+            a = np.full(n, 0x3F80, np.uint16)
+        elif leaf in ("b", "dt_bias", "A_log") and not (leaf == "b" and len(shape) == 2):
+            v = 3.0 if k.endswith(".f.b") else -3.0 if (k.endswith(".dt.b") or leaf == "dt_bias") else 0.0
+            a = SI.st.f32_to_bf16_bits(np.full(n, v, np.float32))
+        else:
+            std = 0.125 if k == "embed" else (0.5 if leaf == "conv" else 1.0 / np.sqrt(shape[-1]))
+            a = SI.st.f32_to_bf16_bits(rng.standard_normal(n, np.float32) * np.float32(std))
+        tensors[k] = a.reshape(shape)
+    return tensors
+
+
+def siladra_section(torch, name, T, iters, warmup, peaks):
+    from . import siladra as SI, seq
+    desc = SI.describe(siladra_config(name))
+    t0 = time.time()
+    rng = np.random.default_rng(0)
+    tensors = siladra_tensors(desc, rng)
+    n_slots = 8
+    m = seq.SeqModel(desc, seq.BF16, n_slots, T + 64, max_rows=T).load(tensors)
+    stream = torch.cuda.ExternalStream(seq.stream_handle(), device=torch.device("cuda", 0))
+    prompt = rng.integers(0, desc["vocab"], T).astype(np.int32)
+    params, mix, dec_bytes = siladra_counts(desc, T)
+    out = {"size": name, "layers": len(desc["layers"]), "params_matmul_per_token": params, "weight_bytes": m.weight_bytes(), "setup_s": round(time.time() - t0, 1)}
+
+    def prefill():
+        m.reset(0)
+        m.step([(0, prompt)], [T - 1])
+    l0 = seq.launch_count()
+    prefill()
+    out["prefill_launches"] = seq.launch_count() - l0
+    ms = _events(torch, stream, prefill, iters, warmup)
+    flops = 2.0 * T * params - 2.0 * (T - 1) * desc["vocab"] * desc["width"] + mix
+    out["prefill"] = {"T": T, "ms": ms, "tokens_per_s": T / ms * 1e3, "tflops": flops / ms * 1e-9, "frac_of_bf16_peak": flops / ms * 1e-9 / peaks["tflops"],
+                      "note": "includes the host->device copy of the prompt and the device->host copy of the last row's logits; experts count top per token"}
+
+    def chunked():                                                # the same prompt in four portions
+        m.reset(0)
+        for i in range(0, T, T // 4):
+            m.step([(0, prompt[i:i + T // 4])], [T // 4 - 1])
+    out["prefill_in_4_portions_ms"] = _events(torch, stream, chunked, max(3, iters // 2), 2)
+    for s in range(n_slots):
+        m.reset(s)
+        m.step_greedy([(s, prompt[: T - 40])])
+    for nseq in (1, 8):
+        slots, steps = list(range(nseq)), 8
+        m.decode(slots, 2)
+        t_ms = []
+        with torch.cuda.stream(stream):
+            for _ in range(3):
+                a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                a.record(stream)
+                m.decode(slots, steps)
+                b.record(stream)
+                torch.cuda.synchronize()
+                t_ms.append(a.elapsed_time(b) / steps)
+        ms = float(np.median(t_ms))
+        out[f"decode_{nseq}"] = {"ms_per_step": ms, "tokens_per_s": nseq / ms * 1e3, "bytes_per_step_one_sequence": dec_bytes, "gbs": dec_bytes / ms * 1e-6,
+                                 "frac_of_hbm_peak": dec_bytes / ms * 1e-6 / peaks["hbm_gbs"],
+                                 "note": "bytes: the weights a step reads (a shared layer's twice); sequences add their states and cached keys"}
+    out["state_bytes_per_slot"] = m.state_bytes_per_slot()
+    m.close()
+    return out
+
+
+def run_siladra(args, root, clock_sampler) -> None:
+    """`--workload siladra`: Siladra at two sizes, Vulosun and Nanotar at the same widths and layer count in the same call."""
+    import torch
+    from . import build, seq
+    build.build(target="seq")
+    torch.cuda.set_device(0)
+    peaks = _peaks(root)
+    seq.init(0)
+    T = 2048
+    iters = max(3, min(args.steps if args.steps != 512 else 5, 20))
+    warm = max(args.warmup if args.warmup != 16 else 3, 3)
+    res = {"siladra": [], "vulosun_same_width": [], "nanotar_same_width": [], "peaks": peaks}
+    with clock_sampler(0) as clk:
+        for name in SILADRA_SIZES:
+            res["siladra"].append(siladra_section(torch, name, T, iters, warm, peaks))
+        for name in VULOSUN_SIZES:
+            res["vulosun_same_width"].append(vulosun_section(torch, name, T, iters, warm, peaks))
+        for name in NANOTAR_SIZES:
+            res["nanotar_same_width"].append(nanotar_section(torch, name, T, iters, warm, peaks))
+    head = res["siladra"][0]
+    print(json.dumps({"metric": "siladra_prefill_tokens_per_s", "value": head["prefill"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+                      "steps": iters, "warmup": warm, "ms_per_step": head["prefill"]["ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+                      "dtype": "bf16 operands, fp32 accumulation; fp32 stream, norms, scores, gates, recurrent state, router", "data": "synthetic",
+                      "config": {"workload": f"Siladra {head['size']} x {head['layers']} layers, random weights: prefill of {T} tokens; decode at that context",
                                  "l2": "weights of a pass exceed L2"},
                       "detail": res, "gpu_launches": head["prefill_launches"], "clocks": clk.summary()}), flush=True)
 

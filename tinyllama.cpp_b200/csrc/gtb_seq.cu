@@ -284,7 +284,7 @@ size_t state_floats(const gtb_seq_branch& d) {
     return d.kind == GTB_MIX_MINGRU ? (size_t)d.dim : (size_t)d.heads * d.dim * d.vdim;
 }
 // chunked mLSTM / delta rule (prompt portions, bf16 mode): rows per chunk, or 0 when the head is too wide for the chunk kernels' shared memory
-int rec_chunk(const gtb_seq_branch& d) { return d.dim <= 128 ? 64 : d.dim <= 256 ? 32 : 0; }
+int rec_chunk(const gtb_seq_branch& d) { return d.kind == GTB_MIX_DELTA && d.vdim > 512 ? 0 : d.dim <= 128 ? 64 : d.dim <= 256 ? 32 : 0; }
 constexpr int GRU_CHUNK = 32;               // rows per chunk of the chunked minGRU scan
 
 // C = (acc ? C : 0) + bias + A . W^T on the library stream; picks the tensor-core kernel, the few-row kernel or the SIMT tile kernel
@@ -739,23 +739,27 @@ RecBranch rec_args(const gtb_seq_model* m, const BranchW& b) {
     return a;
 }
 
-template <int KIND>
-int launch_rec_walk(const PassTables& t, const RecBranch& a, int S, const float* X, int ldx, const float4* G, float* state, float* O) {
+template <int KIND, int RPT>
+void launch_rec_walk_n(const PassTables& t, const RecBranch& a, int S, bool one, const float* X, int ldx, const float* P, int ldp, const float4* G, const float* ms, float* state, float* O) {
     const dim3 grid(S, a.heads, (a.vx + 31) / 32);
-    cudaStream_t st = ctx().stream;
-    if (a.dim <= 32) k_rec_walk<KIND, 4><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
-    else if (a.dim <= 64) k_rec_walk<KIND, 8><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
-    else if (a.dim <= 128) k_rec_walk<KIND, 16><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
-    else if (a.dim <= 256) k_rec_walk<KIND, 32><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
-    else if (a.dim <= 512) k_rec_walk<KIND, 64><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
-    else k_rec_walk<KIND, 128><<<grid, 256, 0, st>>>(t, a, X, ldx, G, state, O);
+    if (one) k_rec_walk<KIND, RPT, true><<<grid, 256, 0, ctx().stream>>>(t, a, X, ldx, P, ldp, G, ms, state, O);
+    else k_rec_walk<KIND, RPT, false><<<grid, 256, 0, ctx().stream>>>(t, a, X, ldx, P, ldp, G, ms, state, O);
+}
+template <int KIND>
+int launch_rec_walk(const PassTables& t, const RecBranch& a, int S, bool one, const float* X, int ldx, const float* P, int ldp, const float4* G, const float* ms, float* state, float* O) {
+    if (a.dim <= 32) launch_rec_walk_n<KIND, 4>(t, a, S, one, X, ldx, P, ldp, G, ms, state, O);
+    else if (a.dim <= 64) launch_rec_walk_n<KIND, 8>(t, a, S, one, X, ldx, P, ldp, G, ms, state, O);
+    else if (a.dim <= 128) launch_rec_walk_n<KIND, 16>(t, a, S, one, X, ldx, P, ldp, G, ms, state, O);
+    else if (a.dim <= 256) launch_rec_walk_n<KIND, 32>(t, a, S, one, X, ldx, P, ldp, G, ms, state, O);
+    else if (a.dim <= 512) launch_rec_walk_n<KIND, 64>(t, a, S, one, X, ldx, P, ldp, G, ms, state, O);
+    else launch_rec_walk_n<KIND, 128>(t, a, S, one, X, ldx, P, ldp, G, ms, state, O);
     GTB_LAUNCHED();
     return GTB_OK;
 }
 template <int KIND, int C, int MT>
 int launch_rec_scan(gtb_seq_model* m, const PassTables& t, const RecBranch& a, int S, size_t ps_qk, size_t ps_w, size_t ps_v, const float* X, int ldx, float* state) {
     const size_t smem = ((size_t)(KIND == REC_DELTA ? 8 : 4) * C * (a.dp + 8) + 2 * (size_t)a.dp * (REC_VS + 8) + 2 * C * (REC_VS + 8)) * 2;
-    static size_t allowed = 48 * 1024;
+    static size_t allowed = 40 * 1024;      // (beside static shared memory)
     if (smem > allowed) { GTB_CUDA(cudaFuncSetAttribute(k_rec_scan<KIND, C, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); allowed = smem; }
     k_rec_scan<KIND, C, MT><<<dim3(S, a.heads, a.vp / REC_VS), 256, smem, ctx().stream>>>(t, a, m->recK, ps_qk, m->recW, ps_w, m->recG, m->recB, X, ldx, m->recV, ps_v, m->recS, state);
     GTB_LAUNCHED();
@@ -774,14 +778,14 @@ template <int KIND, int C>
 int run_rec_chunks(gtb_seq_model* m, const PassTables& t, const RecBranch& a, int R, int S, int n_chunks, float* X, int ldx, float* state) {
     cudaStream_t st = ctx().stream;
     const size_t ps_qk = (size_t)m->max_rows * a.kv_heads * a.dp, ps_w = (size_t)m->max_rows * a.heads * a.dp, ps_v = (size_t)m->max_rows * a.heads * a.vp;
-    const int units = 2 * a.kv_heads + (KIND == REC_MLSTM ? a.heads : 0);
+    const int units = 2 * a.kv_heads + a.heads;
     k_rec_prep<KIND><<<dim3(R, (units + 7) / 8), 256, 0, st>>>(a, X, ldx, m->recQ, m->recK, ps_qk, m->recV, ps_v);
     GTB_LAUNCHED();
     if (KIND == REC_DELTA) {
-        const size_t smem = (size_t)C * (C + 4) * sizeof(float) + 2 * (size_t)C * (a.dp + 8) * 2;
-        static size_t allowed = 48 * 1024;
+        const size_t smem = 2 * (size_t)C * (C + 4) * sizeof(float) + 2 * (size_t)C * (std::max(a.dp, a.vp) + 8) * 2;
+        static size_t allowed = 40 * 1024;      // (beside static shared memory)
         if (smem > allowed) { GTB_CUDA(cudaFuncSetAttribute(k_delta_wy<C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); allowed = smem; }
-        k_delta_wy<C><<<dim3(n_chunks, a.heads), 256, smem, st>>>(t, a, S, m->recK, ps_qk, m->recG, m->recB, X, ldx, m->recW, ps_w);
+        k_delta_wy<C><<<dim3(n_chunks, a.heads), 256, smem, st>>>(t, a, S, m->recK, ps_qk, m->recV, ps_v, m->recG, m->recB, X, ldx, m->recW, ps_w);
         GTB_LAUNCHED();
     }
     int rc = a.dp <= 128 ? launch_rec_scan<KIND, C, 1>(m, t, a, S, ps_qk, ps_w, ps_v, X, ldx, state) : launch_rec_scan<KIND, C, 2>(m, t, a, S, ps_qk, ps_w, ps_v, X, ldx, state);
@@ -808,8 +812,11 @@ int run_rec_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const Ru
     }
     const int C = rec_chunk(b.d);
     const bool chunks = sizeof(OT) == 2 && portions && C > 0;
-    k_rec_gates<KIND><<<dim3(S, a.heads), R == S ? 32 : chunks || R >= 64 * S ? 512 : 64, 0, st>>>(t, a, m->P, l.n1, C, run.mstate[bi], m->recG, chunks ? m->recB : nullptr);
-    GTB_LAUNCHED();
+    const bool one = R == S;                     // every segment is one row: gates and unit lengths inside the walk
+    if (!one) {
+        k_rec_gates<KIND><<<dim3(S, a.heads), R >= 512 * S ? 1024 : chunks || R >= 64 * S ? 256 : 64, 0, st>>>(t, a, m->P, l.n1, C, run.mstate[bi], m->recG, chunks ? m->recB : nullptr);
+        GTB_LAUNCHED();
+    }
     int rc;
     if (chunks) {
         int n_chunks = 0;
@@ -817,22 +824,22 @@ int run_rec_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const Ru
         if ((size_t)n_chunks * a.heads * 2 * a.dp * a.vp > m->rec_s_max) return gtb::fail(GTB_ERR_STATE, "chunk workspace too small");
         rc = C == 64 ? run_rec_chunks<KIND, 64>(m, t, a, R, S, n_chunks, X, ldx, run.state[bi]) : run_rec_chunks<KIND, 32>(m, t, a, R, S, n_chunks, X, ldx, run.state[bi]);
     } else {
-        if (KIND == REC_DELTA) {
+        if (KIND == REC_DELTA && !one) {
             k_rec_unit<<<dim3(R, (2 * a.kv_heads + 3) / 4), 128, 0, st>>>(a, X, ldx);
             GTB_LAUNCHED();
         }
-        rc = launch_rec_walk<KIND>(t, a, S, X, ldx, m->recG, run.state[bi], m->O);
+        rc = launch_rec_walk<KIND>(t, a, S, one, X, ldx, m->P, l.n1, m->recG, run.mstate[bi], run.state[bi], m->O);
     }
     if (rc) return rc;
-    k_rec_post<OT, KIND><<<dim3(R, (a.heads + 3) / 4), 128, 0, st>>>(a, m->O, m->recG, m->P, l.n1, (OT*)m->opC, l.kout_p);
+    k_rec_post<OT, KIND><<<dim3(R, (a.heads + 3) / 4), 128, 0, st>>>(t, a, m->O, one ? nullptr : m->recG, run.mstate[bi], m->P, l.n1, (OT*)m->opC, l.kout_p);
     GTB_LAUNCHED();
     return GTB_OK;
 }
 
-template <typename OT, int LANES, int KS>
+template <typename OT, int LANES, int KS, int TILE>
 int launch_ssm(const PassTables& t, const SsmBranch& a, int S, const float* XC, const float* DT, const float* BC, int ld_bc, const float* P, int ldp, float* state, OT* out, int ld_out) {
     constexpr int NCH = 128 / LANES;
-    k_ssm_scan<OT, LANES, KS><<<dim3(S, (a.inner + NCH - 1) / NCH), 128, 0, ctx().stream>>>(t, a, XC, DT, BC, ld_bc, P, ldp, state, out, ld_out);
+    k_ssm_scan<OT, LANES, KS, TILE><<<dim3(S, (a.inner + NCH - 1) / NCH), 128 + SSM_SERVE, 0, ctx().stream>>>(t, a, XC, DT, BC, ld_bc, P, ldp, state, out, ld_out);
     GTB_LAUNCHED();
     return GTB_OK;
 }
@@ -855,8 +862,8 @@ int run_ssm_branch(gtb_seq_model* m, const PassTables& t, int R, int S, const Ru
     } else rc = product<float>(m, m->ssmBC, b.ld_bc, b.w_dt, b.dt_p, m->ssmDT, a.inner, R, a.inner, b.dt_p, b.d_dtb, 0);    // (the columns behind dt_rank meet zero weights)
     if (rc) return rc;
     OT* out = (OT*)m->opC;
-#define SSM_CASE(N, LN, KS) if (a.state <= N) return launch_ssm<OT, LN, KS>(t, a, S, m->convQ, m->ssmDT, m->ssmBC, b.ld_bc, m->P, l.n1, run.state[bi], out, l.kout_p)
-    SSM_CASE(4, 1, 4); SSM_CASE(8, 2, 4); SSM_CASE(16, 4, 4); SSM_CASE(32, 8, 4); SSM_CASE(64, 16, 4); SSM_CASE(128, 32, 4); SSM_CASE(256, 32, 8);
+#define SSM_CASE(N, LN, KS, TL) if (a.state <= N) return launch_ssm<OT, LN, KS, TL>(t, a, S, m->convQ, m->ssmDT, m->ssmBC, b.ld_bc, m->P, l.n1, run.state[bi], out, l.kout_p)
+    SSM_CASE(4, 1, 4, 8); SSM_CASE(8, 2, 4, 16); SSM_CASE(16, 4, 4, 32); SSM_CASE(32, 8, 4, 32); SSM_CASE(64, 16, 4, 32); SSM_CASE(128, 32, 4, 16); SSM_CASE(256, 32, 8, 8);
 #undef SSM_CASE
     return gtb::fail(GTB_ERR_STATE, "selective scan of %d states per channel", a.state);
 }

@@ -58,10 +58,10 @@ __device__ __forceinline__ void delta_gates(const RecBranch& b, const float* __r
 // differences of two sums keep their precision.  The running maximum is a max-plus scan: rows compose as (F, M) o (F', M') =
 // (F + F', max(M + F', M')).  grid (segments, heads); blockDim a multiple of C (or 32 without Bp).
 template <int KIND>
-__global__ void __launch_bounds__(512) k_rec_gates(PassTables t, RecBranch b, const float* __restrict__ P, int ldp, int C, float* __restrict__ mstate, float4* __restrict__ G,
+__global__ void __launch_bounds__(1024) k_rec_gates(PassTables t, RecBranch b, const float* __restrict__ P, int ldp, int C, float* __restrict__ mstate, float4* __restrict__ G,
                                                    float2* __restrict__ Bp) {
-    __shared__ float sF[16], sM[16];
-    __shared__ double sB[16];
+    __shared__ float sF[32], sM[32];
+    __shared__ double sB[32];
     const int s = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
     const int slot = t.seg_slot[s], row0 = t.seg_row0[s], len = t.seg_len[s];
     float carry = KIND == REC_MLSTM ? mstate[(size_t)slot * b.heads + h] : 0.0f;
@@ -127,12 +127,14 @@ __global__ void __launch_bounds__(128) k_rec_unit(RecBranch b, float* __restrict
 // thread's registers (lane = column); the next row's q, k and v are in flight while the current one is computed.  Raw read-outs go to
 // O [R][heads * vx].  The delta rule needs S^T k before it can write: with r = g S^T k and p = g S^T q from one sweep, u = beta (v - r) and
 // the read-out after the write is p + (k . q) u.
-template <int KIND, int RPT>
-__global__ void __launch_bounds__(256) k_rec_walk(PassTables t, RecBranch b, const float* __restrict__ X, int ldx, const float4* __restrict__ G, float* __restrict__ state,
-                                                  float* __restrict__ O) {
+// ONE: every segment is one row.  The gates are formed here from the projections P (the running maximum mstate is only read: its slices' CTAs share it, and
+// k_rec_post moves it on), and q and k come as they left their convolution -- their lengths are linear factors of r, p, k . q and the write.
+template <int KIND, int RPT, bool ONE>
+__global__ void __launch_bounds__(256) k_rec_walk(PassTables t, RecBranch b, const float* __restrict__ X, int ldx, const float* __restrict__ P, int ldp, const float4* __restrict__ G,
+                                                  const float* __restrict__ mstate, float* __restrict__ state, float* __restrict__ O) {
     constexpr int DP = RPT * 8, NPF = (DP + 255) / 256;
     __shared__ __align__(16) float sq[2][DP], sk[2][DP];
-    __shared__ float part[2][2][8][32], skq[2][8];
+    __shared__ float part[2][2][8][32], skq[2][3][8];
     const int s = blockIdx.x, h = blockIdx.y, hk = h / (b.heads / b.kv_heads), lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
     const int slot = t.seg_slot[s], row0 = t.seg_row0[s], len = t.seg_len[s];
     const int c = blockIdx.z * 32 + lane;
@@ -152,9 +154,17 @@ __global__ void __launch_bounds__(256) k_rec_walk(PassTables t, RecBranch b, con
             kn[j] = i < b.dim ? x[b.k_off + hk * b.dim + i] : 0.0f;
         }
         vn = c < b.vdim ? x[b.v_off + h * b.vdim + c] : 1.0f;
-        gn = G[(size_t)(row0 + n) * b.heads + h];
+        if (!ONE) gn = G[(size_t)(row0 + n) * b.heads + h];
     };
     fetch(0);
+    if (ONE) {
+        if (KIND == REC_MLSTM) {
+            float i, f;
+            mlstm_gates(b, P + (size_t)row0 * ldp, h, i, f);
+            const float m0 = mstate[(size_t)slot * b.heads + h], m = fmaxf(f + m0, i);
+            gn = make_float4(fminf(f + m0 - m, 0.0f), i - m + logf(b.qscale), m, 0.0f);
+        } else delta_gates(b, P + (size_t)row0 * ldp, h, gn.x, gn.y);
+    }
     for (int n = 0; n < len; n++) {
         const int buf = n & 1;
 #pragma unroll
@@ -179,7 +189,7 @@ __global__ void __launch_bounds__(256) k_rec_walk(PassTables t, RecBranch b, con
                 O[(size_t)(row0 + n) * (b.heads * b.vx) + h * b.vx + c] = o;
             }
         } else {
-            float r = 0.0f, kq = 0.0f;
+            float r = 0.0f, kq = 0.0f, k2 = 0.0f, q2 = 0.0f;
 #pragma unroll
             for (int j = 0; j < RPT; j++) {
                 const float kk = sk[buf][wid * RPT + j], qq = sq[buf][wid * RPT + j];
@@ -187,17 +197,28 @@ __global__ void __launch_bounds__(256) k_rec_walk(PassTables t, RecBranch b, con
                 r = fmaf(S[j], kk, r);
                 o = fmaf(S[j], qq, o);
                 kq = fmaf(kk, qq, kq);
+                if (ONE) { k2 = fmaf(kk, kk, k2); q2 = fmaf(qq, qq, q2); }
             }
             part[buf][0][wid][lane] = r;
             part[buf][1][wid][lane] = o;
-            if (lane == 0) skq[buf][wid] = kq;
+            if (lane == 0) { skq[buf][0][wid] = kq; skq[buf][1][wid] = k2; skq[buf][2][wid] = q2; }
             __syncthreads();
-            r = o = kq = 0.0f;
+            r = o = kq = k2 = q2 = 0.0f;
 #pragma unroll
-            for (int k = 0; k < 8; k++) { r += part[buf][0][k][lane]; o += part[buf][1][k][lane]; kq += skq[buf][k]; }
-            const float u = w * (v - r);
+            for (int k = 0; k < 8; k++) {
+                r += part[buf][0][k][lane]; o += part[buf][1][k][lane]; kq += skq[buf][0][k];
+                if (ONE) { k2 += skq[buf][1][k]; q2 += skq[buf][2][k]; }
+            }
+            float u, ks = 1.0f;
+            if (ONE) {
+                ks = 1.0f / sqrtf(k2 + 1e-6f);
+                const float qs = b.qscale / sqrtf(q2 + 1e-6f);
+                r *= ks; o *= qs; kq *= ks * qs;
+            }
+            u = w * (v - r);
+            const float ku = ks * u;
 #pragma unroll
-            for (int j = 0; j < RPT; j++) S[j] = fmaf(sk[buf][wid * RPT + j], u, S[j]);
+            for (int j = 0; j < RPT; j++) S[j] = fmaf(sk[buf][wid * RPT + j], ku, S[j]);
             if (wid == 0 && ok) O[(size_t)(row0 + n) * (b.heads * b.vx) + h * b.vx + c] = fmaf(kq, u, o);
         }
     }
@@ -207,15 +228,28 @@ __global__ void __launch_bounds__(256) k_rec_walk(PassTables t, RecBranch b, con
 }
 
 // Output of a (row, head), a warp each: mLSTM o = O / (max(|n . q|, exp(-m)) + 1e-6); both: o / sqrt(mean(o^2) + eps) * norm * gate
-// (mLSTM: logistic, delta rule: silu) -> out-projection operand
+// (mLSTM: logistic, delta rule: silu) -> out-projection operand.  G null (mLSTM, every segment one row): the running maximum is formed here and moved on.
 template <typename OT, int KIND>
-__global__ void __launch_bounds__(128) k_rec_post(RecBranch b, const float* __restrict__ O, const float4* __restrict__ G, const float* __restrict__ P, int ldp,
-                                                  OT* __restrict__ out, int ld_out) {
+__global__ void __launch_bounds__(128) k_rec_post(PassTables t, RecBranch b, const float* __restrict__ O, const float4* __restrict__ G, float* __restrict__ mstate,
+                                                  const float* __restrict__ P, int ldp, OT* __restrict__ out, int ld_out) {
     const int r = blockIdx.x, lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
     for (int h = blockIdx.y * nw + wid; h < b.heads; h += gridDim.y * nw) {
         const float* o = O + (size_t)r * (b.heads * b.vx) + h * b.vx;
         float dn = 1.0f;
-        if (KIND == REC_MLSTM) dn = 1.0f / (fmaxf(fabsf(o[b.vdim]), expf(-G[(size_t)r * b.heads + h].z)) + 1e-6f);
+        if (KIND == REC_MLSTM) {
+            float m;
+            if (G) m = G[(size_t)r * b.heads + h].z;
+            else {
+                const int slot = t.seg_slot[t.row_seg[r]];
+                float i, f;
+                mlstm_gates(b, P + (size_t)r * ldp, h, i, f);
+                float* ms = mstate + (size_t)slot * b.heads + h;
+                m = fmaxf(f + *ms, i);
+                __syncwarp();
+                if (lane == 0 && !t.slots[slot].stopped) *ms = m;
+            }
+            dn = 1.0f / (fmaxf(fabsf(o[b.vdim]), expf(-m)) + 1e-6f);
+        }
         float ss = 0.0f;
         for (int i = lane; i < b.vdim; i += 32) { const float v = o[i] * dn; ss += v * v; }
         const float sc = dn * b.out_scale / sqrtf(warp_sum(ss) / (float)b.vdim + b.eps);
@@ -241,9 +275,9 @@ __global__ void __launch_bounds__(256) k_rec_prep(RecBranch b, const float* __re
                                                   bf16* __restrict__ VPn, size_t ps_v) {
     const int r = blockIdx.x, lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
     const float* x = X + (size_t)r * ldx;
-    const int units = 2 * b.kv_heads + (KIND == REC_MLSTM ? b.heads : 0);
+    const int units = 2 * b.kv_heads + b.heads;
     for (int u = blockIdx.y * nw + wid; u < units; u += gridDim.y * nw) {
-        if (u >= 2 * b.kv_heads) {           // values and the column of ones
+        if (u >= 2 * b.kv_heads) {           // values, and the column of ones of a normaliser
             const int h = u - 2 * b.kv_heads;
             bf16* d = VPn + ((size_t)r * b.heads + h) * b.vp;
             for (int i = lane * 2; i < b.vp; i += 64) {
@@ -277,46 +311,52 @@ __global__ void __launch_bounds__(256) k_rec_prep(RecBranch b, const float* __re
 }
 
 // planes of rows [row0, row0 + C) (rows from L on: zeros), columns [0, w) of a head -> shared memory [2][C][ld]; w a multiple of 8
+// (a warp covers 1, 2 or 4 rows at a time)
 __device__ __forceinline__ void rec_stage(uint32_t dst, int ld, int C, const bf16* __restrict__ src, size_t ps, size_t row_ld, int L, int w) {
-    const int per = w / 8;
-    for (int e = threadIdx.x; e < 2 * C * per; e += blockDim.x) {
-        const int pl = e / (C * per), rem = e % (C * per), r = rem / per, c8 = (rem % per) * 8;
-        sa_cp16(dst + (uint32_t)(((pl * C + r) * ld + c8) * 2), r < L ? (const void*)(src + pl * ps + (size_t)r * row_ld + c8) : (const void*)src, r < L);
+    const int per = w >> 3, sh = per <= 8 ? 3 : per <= 16 ? 4 : 5, lane = threadIdx.x & 31, piece = lane & ((1 << sh) - 1), rows = 32 >> sh;
+    for (int r = (threadIdx.x >> 5) * rows + (lane >> sh); r < 2 * C; r += (blockDim.x >> 5) * rows) {
+        const int pl = r >= C, rr = r - pl * C;
+        const bool on = rr < L;
+        for (int c = piece; c < per; c += 1 << sh)
+            sa_cp16(dst + (uint32_t)((r * ld + c * 8) * 2), on ? (const void*)(src + pl * ps + (size_t)rr * row_ld + c * 8) : (const void*)src, on);
     }
 }
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// grid (chunks, heads), 256 threads.  The chunk's A from k's planes on tensor cores, then forward substitution: a thread per column of
-// [W | U'] keeps the column's C values in registers, A's rows come as broadcast reads.
+// grid (chunks, heads), 256 threads.  The chunk's A from k's planes on tensor cores; T = (I + A)^-1 in fp32 by blocks of 16 rows -- the diagonal blocks by
+// forward substitution (a thread per column), T_ij = -T_ii sum_k A_ik T_kj below them, one block diagonal after the other; then W = (T diag(beta e^b)) K
+// and U' = (T diag(beta)) V on tensor cores, T's scaled columns split into planes on the way into the A fragments.
+// VPn: planes of v; U' goes to X's v columns.
 template <int C>
-__global__ void __launch_bounds__(256) k_delta_wy(PassTables t, RecBranch b, int S, const bf16* __restrict__ KP, size_t ps_qk, const float4* __restrict__ G,
-                                                  const float2* __restrict__ Bp, float* __restrict__ X, int ldx, bf16* __restrict__ WP, size_t ps_w) {
+__global__ void __launch_bounds__(256, 2) k_delta_wy(PassTables t, RecBranch b, int S, const bf16* __restrict__ KP, size_t ps_qk, const bf16* __restrict__ VPn, size_t ps_v,
+                                                     const float4* __restrict__ G, const float2* __restrict__ Bp, float* __restrict__ X, int ldx, bf16* __restrict__ WP, size_t ps_w) {
     extern __shared__ __align__(16) unsigned char rc_raw[];
-    __shared__ float sbeta[C], sbh[C], sbl[C];
-    constexpr int LA = C + 4;
+    __shared__ float sbeta[C], sbeb[C], sbh[C], sbl[C];
+    constexpr int LA = C + 4, NB = C / 16;
     int seg, ck;
     if (!ret_find_chunk(t, S, C, blockIdx.x, seg, ck)) return;
-    const int h = blockIdx.y, hk = h / (b.heads / b.kv_heads), LK = b.dp + 8;
+    const int h = blockIdx.y, hk = h / (b.heads / b.kv_heads), LK = b.dp + 8, LV = b.vp + 8;
     const int row0 = t.seg_row0[seg] + ck * C, L = min(C, t.seg_len[seg] - ck * C);
     float* sA = reinterpret_cast<float*>(rc_raw);                // [C][LA]
-    bf16* sk = reinterpret_cast<bf16*>(sA + C * LA);             // [2][C][LK]
+    float* sT = sA + C * LA;                                     // [C][LA]; block (i, j) also holds sum_k A_ik T_kj on its way to T_ij
+    bf16* sk = reinterpret_cast<bf16*>(sT + C * LA);             // [2][C][max(LK, LV)]: k, then v
     const uint32_t sk_a = (uint32_t)__cvta_generic_to_shared(sk);
     rec_stage(sk_a, LK, C, KP + ((size_t)row0 * b.kv_heads + hk) * b.dp, ps_qk, (size_t)b.kv_heads * b.dp, L, b.dp);
     cp_commit();
     for (int r = threadIdx.x; r < C; r += 256) {
         float2 bb = make_float2(0.0f, 0.0f);
-        if (r < L) bb = Bp[(size_t)(row0 + r) * b.heads + h];
-        sbeta[r] = r < L ? G[(size_t)(row0 + r) * b.heads + h].y : 0.0f;
-        sbh[r] = bb.x; sbl[r] = bb.y;
+        float be = 0.0f;
+        if (r < L) { bb = Bp[(size_t)(row0 + r) * b.heads + h]; be = G[(size_t)(row0 + r) * b.heads + h].y; }
+        sbeta[r] = be; sbh[r] = bb.x; sbl[r] = bb.y; sbeb[r] = be * expf(bb.x + bb.y);
     }
     cp_wait<0>();
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
-    for (int tile = warp; tile < (C / 16) * (C / 16); tile += 8) {
-        const int mt = tile / (C / 16), nt = tile % (C / 16);
+    for (int tile = warp; tile < NB * NB; tile += 8) {
+        const int mt = tile / NB, nt = tile % NB;
         if (nt > mt) continue;                                   // above the diagonal nothing is read
-        float acc[2][4] = {};
+        float acc[2][4] = {}, acx[2][4] = {};
         for (int kk = 0; kk < b.dp / 16; kk++) {
             uint32_t a[2][4], w[2][4];
 #pragma unroll
@@ -327,8 +367,8 @@ __global__ void __launch_bounds__(256) k_delta_wy(PassTables t, RecBranch b, int
 #pragma unroll
             for (int n = 0; n < 2; n++) {
                 sa_mma(acc[n], a[0], w[0][2 * n], w[0][2 * n + 1]);
-                sa_mma(acc[n], a[0], w[1][2 * n], w[1][2 * n + 1]);
-                sa_mma(acc[n], a[1], w[0][2 * n], w[0][2 * n + 1]);
+                sa_mma(acx[n], a[0], w[1][2 * n], w[1][2 * n + 1]);
+                sa_mma(acx[n], a[1], w[0][2 * n], w[0][2 * n + 1]);
             }
         }
 #pragma unroll
@@ -336,42 +376,105 @@ __global__ void __launch_bounds__(256) k_delta_wy(PassTables t, RecBranch b, int
 #pragma unroll
             for (int x = 0; x < 4; x++) {
                 const int tt = mt * 16 + gq + (x >= 2 ? 8 : 0), ss = nt * 16 + n * 8 + tq * 2 + (x & 1);
-                sA[tt * LA + ss] = (ss < tt && tt < L) ? sbeta[tt] * expf((sbh[tt] - sbh[ss]) + (sbl[tt] - sbl[ss])) * acc[n][x] : 0.0f;
+                sA[tt * LA + ss] = (ss < tt && tt < L) ? sbeta[tt] * expf((sbh[tt] - sbh[ss]) + (sbl[tt] - sbl[ss])) * (acc[n][x] + acx[n][x]) : 0.0f;
             }
     }
     __syncthreads();
-    for (int col = threadIdx.x; col < b.dp + b.vdim; col += 256) {
-        float x[C];
-        const bool is_w = col < b.dp;
-        float* xv = X + (size_t)row0 * ldx + b.v_off + h * b.vdim + (col - b.dp);
+    if (threadIdx.x < C) {                                       // diagonal blocks
+        const int b0 = (threadIdx.x >> 4) * 16, col = threadIdx.x & 15;
+        float x[16];
 #pragma unroll
-        for (int r = 0; r < C; r++) {
-            if (is_w) x[r] = sbeta[r] * expf(sbh[r]) * (__bfloat162float(sk[r * LK + col]) + __bfloat162float(sk[(C + r) * LK + col]));
-            else x[r] = r < L ? sbeta[r] * xv[(size_t)r * ldx] : 0.0f;
+        for (int r = 0; r < 16; r++) {
+            float a0 = r == col ? 1.0f : 0.0f;
+#pragma unroll
+            for (int q = 0; q < r; q++) a0 = fmaf(-sA[(b0 + r) * LA + b0 + q], x[q], a0);
+            x[r] = a0;
+            sT[(b0 + r) * LA + b0 + col] = a0;
         }
+    }
+    __syncthreads();
 #pragma unroll
-        for (int r = 1; r < C; r++) {
-            float a0 = x[r], a1 = 0.0f;
+    for (int d = 1; d < NB; d++) {                               // blocks (j + d, j)
+        const int r = threadIdx.x >> 4, c = threadIdx.x & 15;
 #pragma unroll
-            for (int q = 0; q < (r + 3) / 4; q++) {              // entries from r on are zero
-                const float4 a4 = *reinterpret_cast<const float4*>(sA + r * LA + q * 4);
-                a0 = fmaf(-a4.x, x[q * 4], a0);
-                if (q * 4 + 1 < r) a1 = fmaf(-a4.y, x[q * 4 + 1], a1);
-                if (q * 4 + 2 < r) a0 = fmaf(-a4.z, x[q * 4 + 2], a0);
-                if (q * 4 + 3 < r) a1 = fmaf(-a4.w, x[q * 4 + 3], a1);
+        for (int j = 0; j + d < NB; j++) {
+            const int i = j + d;
+            float a0 = 0.0f, a1 = 0.0f;
+            for (int k = j * 16; k < i * 16; k += 2) { a0 = fmaf(sA[(i * 16 + r) * LA + k], sT[k * LA + j * 16 + c], a0); a1 = fmaf(sA[(i * 16 + r) * LA + k + 1], sT[(k + 1) * LA + j * 16 + c], a1); }
+            sT[(i * 16 + r) * LA + j * 16 + c] = a0 + a1;
+        }
+        __syncthreads();
+        float v[NB];
+#pragma unroll
+        for (int j = 0; j + d < NB; j++) {
+            const int i = j + d;
+            float a0 = 0.0f;
+#pragma unroll
+            for (int k = 0; k < 16; k++) a0 = fmaf(sT[(i * 16 + r) * LA + i * 16 + k], sT[(i * 16 + k) * LA + j * 16 + c], a0);
+            v[j] = -a0;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int j = 0; j + d < NB; j++) sT[((j + d) * 16 + r) * LA + j * 16 + c] = v[j];
+        __syncthreads();
+    }
+    const int mt = warp % NB, part = warp / NB, n_part = 8 / NB;  // this warp's 16 rows and its share of the columns
+#pragma unroll
+    for (int pass = 0; pass < 2; pass++) {                       // W, then U'
+        const int LB = pass ? LV : LK, nw16 = (pass ? b.vp : b.dp) / 16;
+        if (pass) {
+            __syncthreads();                                     // k's planes have been read
+            rec_stage(sk_a, LV, C, VPn + ((size_t)row0 * b.heads + h) * b.vp, ps_v, (size_t)b.heads * b.vp, L, b.vp);
+            cp_commit();
+        }
+        uint32_t ah[NB][4], al[NB][4];
+#pragma unroll
+        for (int kk = 0; kk < NB; kk++) {
+            if (kk > mt) continue;
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int rr = mt * 16 + gq + (e & 1) * 8, c = kk * 16 + tq * 2 + (e >> 1) * 8;
+                const float* sc = pass ? sbeta : sbeb;
+                const bool low = kk < mt || c <= rr, low1 = kk < mt || c + 1 <= rr;
+                split2_pack(low ? sT[rr * LA + c] * sc[c] : 0.0f, low1 ? sT[rr * LA + c + 1] * sc[c + 1] : 0.0f, ah[kk][e], al[kk][e]);
             }
-            x[r] = a0 + a1;
         }
-        bf16* wd = WP + ((size_t)row0 * b.heads + h) * b.dp + col;
+        if (pass) { cp_wait<0>(); __syncthreads(); }
+        for (int n2 = part; n2 < nw16; n2 += n_part) {
+            float acc[2][4] = {}, acx[2][4] = {};
 #pragma unroll
-        for (int r = 0; r < C; r++) {
-            if (r >= L) break;
-            if (is_w) {
-                bf16 hi, lo;
-                split2(x[r], hi, lo);
-                wd[(size_t)r * b.heads * b.dp] = hi;
-                wd[ps_w + (size_t)r * b.heads * b.dp] = lo;
-            } else xv[(size_t)r * ldx] = x[r];
+            for (int kk = 0; kk < NB; kk++) {
+                if (kk > mt) continue;
+                uint32_t w[2][4];
+#pragma unroll
+                for (int pl = 0; pl < 2; pl++)
+                    sa_ldsm_x4_t(sk_a + (uint32_t)(((pl * C + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LB + n2 * 16 + (lane >> 4) * 8) * 2), w[pl][0], w[pl][1], w[pl][2], w[pl][3]);
+#pragma unroll
+                for (int n = 0; n < 2; n++) {
+                    sa_mma(acc[n], ah[kk], w[0][2 * n], w[0][2 * n + 1]);
+                    sa_mma(acx[n], ah[kk], w[1][2 * n], w[1][2 * n + 1]);
+                    sa_mma(acx[n], al[kk], w[0][2 * n], w[0][2 * n + 1]);
+                }
+            }
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int hf = 0; hf < 2; hf++) {
+                    const int rr = mt * 16 + gq + hf * 8, c = n2 * 16 + n * 8 + tq * 2;
+                    if (rr >= L) continue;
+                    const float v0 = acc[n][2 * hf] + acx[n][2 * hf], v1 = acc[n][2 * hf + 1] + acx[n][2 * hf + 1];
+                    if (pass == 0) {
+                        uint32_t hi, lo;
+                        split2_pack(v0, v1, hi, lo);
+                        bf16* wd = WP + ((size_t)(row0 + rr) * b.heads + h) * b.dp + c;
+                        *reinterpret_cast<uint32_t*>(wd) = hi;
+                        *reinterpret_cast<uint32_t*>(wd + ps_w) = lo;
+                    } else {
+                        float* xv = X + (size_t)(row0 + rr) * ldx + b.v_off + h * b.vdim + c;
+                        if (c < b.vdim) xv[0] = v0;
+                        if (c + 1 < b.vdim) xv[1] = v1;
+                    }
+                }
         }
     }
 }
@@ -415,15 +518,35 @@ __global__ void __launch_bounds__(256) k_rec_scan(PassTables t, RecBranch b, con
         const int row0 = t.seg_row0[seg] + ck * C, L = min(C, len - ck * C);
         rec_stage(sk_a + (uint32_t)(st * 2 * C * LK * 2), LK, C, KP + ((size_t)row0 * b.kv_heads + hk) * b.dp, ps_qk, (size_t)b.kv_heads * b.dp, L, b.dp);
         if (KIND == REC_DELTA) rec_stage(sw_a + (uint32_t)(st * 2 * C * LK * 2), LK, C, WP + ((size_t)row0 * b.heads + h) * b.dp, ps_w, (size_t)b.heads * b.dp, L, b.dp);
-        for (int r = threadIdx.x; r < C; r += 256) {
-            float2 bb = make_float2(0.0f, 0.0f);
-            float lw = 0.0f;
-            if (r < L) { bb = Bp[(size_t)(row0 + r) * b.heads + h]; if (KIND == REC_MLSTM) lw = G[(size_t)(row0 + r) * b.heads + h].y; }
-            sbh[st][r] = bb.x; sbl[st][r] = bb.y; slw[st][r] = lw;
-        }
         cp_commit();
     };
+    // gates of one chunk and this thread's elements of u of the next one wait in registers: for the delta rule those of its U tile (warp -> 16 rows x 8
+    // columns), otherwise rows of [v | 1]
+    float2 gb = make_float2(0.0f, 0.0f);
+    float glw = 0.0f, un[4];
+    const int ut = (warp >> 1) * 16 + gq, uc = c0 + (warp & 1) * 8 + tq * 2;
+    const bool has_u = (warp >> 1) * 16 < C;
+    auto fetch_gates = [&](int ck) {
+        const int r = ck * C + (int)threadIdx.x;
+        if ((int)threadIdx.x >= C) return;
+        gb = make_float2(0.0f, 0.0f);
+        glw = 0.0f;
+        if (r < len) { const size_t at = (size_t)(t.seg_row0[seg] + r) * b.heads + h; gb = Bp[at]; if (KIND == REC_MLSTM) glw = G[at].y; }
+    };
+    auto put_gates = [&](int st) { if ((int)threadIdx.x < C) { sbh[st][threadIdx.x] = gb.x; sbl[st][threadIdx.x] = gb.y; slw[st][threadIdx.x] = glw; } };
+    auto fetch_u = [&](int ck) {
+#pragma unroll
+        for (int x = 0; x < 4; x++) {
+            const int r = ck * C + ut + (x >= 2 ? 8 : 0), c = uc + (x & 1);
+            un[x] = 0.0f;
+            if (has_u && r < len) un[x] = c < b.vdim ? X[(size_t)(t.seg_row0[seg] + r) * ldx + b.v_off + h * b.vdim + c] : (c < b.vx ? 1.0f : 0.0f);
+        }
+    };
     stage(0, 0);
+    fetch_gates(0);
+    put_gates(0);
+    fetch_gates(1);
+    fetch_u(0);
     for (int ck = 0; ck < n_ck; ck++) {
         const int st = ck & 1, row0 = t.seg_row0[seg] + ck * C, L = min(C, len - ck * C);
         bf16* sp = SP + ((size_t)(first + ck) * b.heads + h) * 2 * b.dp * b.vp + c0;
@@ -443,23 +566,19 @@ __global__ void __launch_bounds__(256) k_rec_scan(PassTables t, RecBranch b, con
                     *reinterpret_cast<uint32_t*>(sp + ((size_t)b.dp + d) * b.vp + c) = lo;
                 }
         }
-        // this thread's elements of u: for the delta rule those of its U tile (warp -> 16 rows x 8 columns), otherwise rows of [v | 1]
-        float u[4];
-        const int ut = (warp >> 1) * 16 + gq, uc = c0 + (warp & 1) * 8 + tq * 2;
-        const bool has_u = (warp >> 1) * 16 < C;
-#pragma unroll
-        for (int x = 0; x < 4; x++) {
-            const int r = ut + (x >= 2 ? 8 : 0), c = uc + (x & 1);
-            u[x] = 0.0f;
-            if (has_u && r < L) u[x] = c < b.vdim ? X[(size_t)(row0 + r) * ldx + b.v_off + h * b.vdim + c] : (c < b.vx ? 1.0f : 0.0f);
-        }
+        float u[4] = {un[0], un[1], un[2], un[3]};
         cp_wait<0>();
         __syncthreads();
-        if (ck + 1 < n_ck) stage(st ^ 1, ck + 1);                            // its last readers passed the barrier above
+        if (ck + 1 < n_ck) {                                                 // its last readers passed the barrier above
+            stage(st ^ 1, ck + 1);
+            put_gates(st ^ 1);
+            fetch_gates(ck + 2);
+            fetch_u(ck + 1);
+        }
         const float bLh = sbh[st][L - 1], bLl = sbl[st][L - 1];
         if (has_u) {
             if (KIND == REC_DELTA) {
-                float ws[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+                float ws[3][4] = {};
                 const int m0 = (warp >> 1) * 16, n8 = (warp & 1) * 8;
                 for (int kk = 0; kk < nmt; kk++) {
                     uint32_t a[2][4], s0[2], s1[2];
@@ -468,12 +587,12 @@ __global__ void __launch_bounds__(256) k_rec_scan(PassTables t, RecBranch b, con
                         sa_ldsm_x4(sw_a + (uint32_t)((((st * 2 + pl) * C + m0 + (lane & 15)) * LK + kk * 16 + (lane >> 4) * 8) * 2), a[pl][0], a[pl][1], a[pl][2], a[pl][3]);
                     // hi and lo of the state's 16 rows at once: lanes 0 - 15 address the hi plane, 16 - 31 the lo plane
                     sa_ldsm_x4_t(sS_a + (uint32_t)((((lane >> 4) * b.dp + kk * 16 + (lane & 15)) * LS + n8) * 2), s0[0], s0[1], s1[0], s1[1]);
-                    sa_mma(ws, a[0], s0[0], s0[1]);
-                    sa_mma(ws, a[0], s1[0], s1[1]);
-                    sa_mma(ws, a[1], s0[0], s0[1]);
+                    sa_mma(ws[0], a[0], s0[0], s0[1]);
+                    sa_mma(ws[1], a[0], s1[0], s1[1]);
+                    sa_mma(ws[2], a[1], s0[0], s0[1]);
                 }
 #pragma unroll
-                for (int x = 0; x < 4; x++) u[x] = ut + (x >= 2 ? 8 : 0) < L ? u[x] - ws[x] : 0.0f;
+                for (int x = 0; x < 4; x++) u[x] = ut + (x >= 2 ? 8 : 0) < L ? u[x] - (ws[0][x] + (ws[1][x] + ws[2][x])) : 0.0f;
             }
 #pragma unroll
             for (int hf = 0; hf < 2; hf++) {
@@ -493,12 +612,13 @@ __global__ void __launch_bounds__(256) k_rec_scan(PassTables t, RecBranch b, con
         }
         __syncthreads();
         const float dec = expf(bLh + bLl);
+        float acx[MT][2][4];                                                 // the products with a lo plane
 #pragma unroll
         for (int i = 0; i < MT; i++)
 #pragma unroll
             for (int n = 0; n < 2; n++)
 #pragma unroll
-                for (int x = 0; x < 4; x++) acc[i][n][x] *= dec;
+                for (int x = 0; x < 4; x++) { acc[i][n][x] *= dec; acx[i][n][x] = 0.0f; }
 #pragma unroll
         for (int kk = 0; kk < C / 16; kk++) {
             uint32_t w[2][4];
@@ -516,11 +636,17 @@ __global__ void __launch_bounds__(256) k_rec_scan(PassTables t, RecBranch b, con
 #pragma unroll
                 for (int n = 0; n < 2; n++) {
                     sa_mma(acc[i][n], a[0], w[0][2 * n], w[0][2 * n + 1]);
-                    sa_mma(acc[i][n], a[0], w[1][2 * n], w[1][2 * n + 1]);
-                    sa_mma(acc[i][n], a[1], w[0][2 * n], w[0][2 * n + 1]);
+                    sa_mma(acx[i][n], a[0], w[1][2 * n], w[1][2 * n + 1]);
+                    sa_mma(acx[i][n], a[1], w[0][2 * n], w[0][2 * n + 1]);
                 }
             }
         }
+#pragma unroll
+        for (int i = 0; i < MT; i++)
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int x = 0; x < 4; x++) acc[i][n][x] += acx[i][n][x];
     }
     if (t.slots[slot].stopped) return;
 #pragma unroll
@@ -664,20 +790,74 @@ struct SsmBranch {
     const float *A_log, *D;                  // [inner][state], [inner]
     float out_scale;
 };
-// Walks the rows of a segment for 128 / LANES channels: LANES neighbouring threads share a channel, KS of its states in each thread's
-// registers.  Rows come in tiles of SSM_TILE through shared memory (step size, step size times input, output share and gate per channel; B and C
-// of the row), so the chain per row is one multiply-add per state.  XC [R][inner]: input behind its convolution; DT [R][inner]: step sizes before the
-// softplus; BC [R][ld_bc]: columns dt_rank.. are B, then C.
-constexpr int SSM_TILE = 16;
-template <typename OT, int LANES, int KS>
-__global__ void __launch_bounds__(128) k_ssm_scan(PassTables t, SsmBranch b, const float* __restrict__ XC, const float* __restrict__ DT, const float* __restrict__ BC, int ld_bc,
+// Walks the rows of a segment for 128 / LANES channels.  Threads 0 .. 127 scan: LANES neighbouring ones share a channel, KS of its states in each
+// thread's registers, so the chain per row is one multiply-add per state.  The other SSM_SERVE threads serve them, a tile of TILE rows ahead and one behind: step
+// sizes and inputs, B and C of the next tile into shared memory, outputs of the previous tile out of it (one barrier per tile).
+// XC [R][inner]: input behind its convolution; DT [R][inner]: step sizes before the softplus; BC [R][ld_bc]: columns dt_rank.. are B, then C.
+constexpr int SSM_SERVE = 384;
+template <typename OT, int LANES, int KS, int TILE>
+__global__ void __launch_bounds__(128 + SSM_SERVE) k_ssm_scan(PassTables t, SsmBranch b, const float* __restrict__ XC, const float* __restrict__ DT, const float* __restrict__ BC, int ld_bc,
                                                   const float* __restrict__ P, int ldp, float* __restrict__ state, OT* __restrict__ out, int ld_out) {
-    constexpr int NCH = 128 / LANES, NSP = LANES * KS;
-    __shared__ __align__(16) float sB[SSM_TILE][NSP], sC[SSM_TILE][NSP];
-    __shared__ float2 sdx[SSM_TILE][NCH];                 // {dt, dt x}
-    __shared__ float sy[SSM_TILE][NCH + 1];
-    const int s = blockIdx.x, ch0 = blockIdx.y * NCH, ci = threadIdx.x / LANES, li = threadIdx.x % LANES, ch = ch0 + ci;
-    const int slot = t.seg_slot[s], row0 = t.seg_row0[s], len = t.seg_len[s];
+    constexpr int NCH = 128 / LANES, NSP = LANES * KS, NE = (TILE * NCH + SSM_SERVE - 1) / SSM_SERVE;      // NE: (row, channel) pairs of a tile per serving thread
+    __shared__ __align__(16) float sB[2][TILE][NSP], sC[2][TILE][NSP];
+    __shared__ float2 sdx[2][TILE][NCH];                  // {dt, dt x}
+    __shared__ float sy[2][TILE][NCH + 1];
+    const int s = blockIdx.x, ch0 = blockIdx.y * NCH;
+    const int slot = t.seg_slot[s], row0 = t.seg_row0[s], len = t.seg_len[s], n_t = (len + TILE - 1) / TILE;
+    if (threadIdx.x >= 128) {
+        const int tid = threadIdx.x - 128;
+        auto fill = [&](int it) {
+            const int n0 = it * TILE, nt = min(TILE, len - n0), buf = it & 1;
+            float x[NE], z[NE];
+#pragma unroll
+            for (int i = 0; i < NE; i++) {
+                const int e = tid + i * SSM_SERVE, r = e / NCH, c = ch0 + e % NCH;
+                const bool on = r < nt && c < b.inner;
+                const size_t at = (size_t)(row0 + n0 + r) * b.inner + c;
+                z[i] = on ? DT[at] : 0.0f;
+                x[i] = on ? XC[at] : 0.0f;
+            }
+            for (int e = tid; e < TILE * NSP; e += SSM_SERVE) {
+                const int r = e / NSP, n = e % NSP;
+                const float* p = BC + (size_t)(row0 + n0 + r) * ld_bc + b.dt_rank;
+                const bool on = r < nt && n < b.state;
+                sB[buf][r][n] = on ? p[n] : 0.0f;
+                sC[buf][r][n] = on ? p[b.state + n] : 0.0f;
+            }
+#pragma unroll
+            for (int i = 0; i < NE; i++) {
+                const int e = tid + i * SSM_SERVE;
+                const float dt = softplus_(z[i]);
+                if (e < TILE * NCH) sdx[buf][e / NCH][e % NCH] = make_float2(dt, dt * x[i]);
+            }
+        };
+        auto drain = [&](int it) {
+            const int n0 = it * TILE, nt = min(TILE, len - n0), buf = it & 1;
+            float x[NE], z[NE];
+#pragma unroll
+            for (int i = 0; i < NE; i++) {
+                const int e = tid + i * SSM_SERVE, r = e / NCH, c = ch0 + e % NCH;
+                const bool on = r < nt && c < b.inner;
+                x[i] = on ? b.D[c] * XC[(size_t)(row0 + n0 + r) * b.inner + c] : 0.0f;
+                z[i] = on ? P[(size_t)(row0 + n0 + r) * ldp + b.z_off + c] : 0.0f;
+            }
+#pragma unroll
+            for (int i = 0; i < NE; i++) {
+                const int e = tid + i * SSM_SERVE, r = e / NCH, c = ch0 + e % NCH;
+                if (r < nt && c < b.inner) out[(size_t)(row0 + n0 + r) * ld_out + b.a_off + c] = cvt<OT>((sy[buf][r][e % NCH] + x[i]) * (sizeof(OT) == 2 ? __fdividef(z[i], 1.0f + __expf(-z[i])) : silu_(z[i])) * b.out_scale);
+            }
+        };
+        fill(0);
+        __syncthreads();
+        for (int it = 0; it < n_t; it++) {
+            if (it + 1 < n_t) fill(it + 1);
+            if (it > 0) drain(it - 1);
+            __syncthreads();
+        }
+        drain(n_t - 1);
+        return;
+    }
+    const int ci = threadIdx.x / LANES, li = threadIdx.x % LANES, ch = ch0 + ci;
     const bool ok = ch < b.inner;
     float* gs = state + ((size_t)slot * b.inner + (ok ? ch : 0)) * b.state;
     float S[KS], A[KS];
@@ -689,45 +869,30 @@ __global__ void __launch_bounds__(128) k_ssm_scan(PassTables t, SsmBranch b, con
         A[k] = in ? -expf(b.A_log[(size_t)ch * b.state + n]) : 0.0f;
         if (sizeof(OT) == 2) A[k] *= 1.4426950408889634f;
     }
-    for (int n0 = 0; n0 < len; n0 += SSM_TILE) {
-        const int nt = min(SSM_TILE, len - n0);
-        for (int e = threadIdx.x; e < nt * NSP; e += 128) {
-            const int r = e / NSP, n = e % NSP;
-            const float* p = BC + (size_t)(row0 + n0 + r) * ld_bc + b.dt_rank;
-            sB[r][n] = n < b.state ? p[n] : 0.0f;
-            sC[r][n] = n < b.state ? p[b.state + n] : 0.0f;
-        }
-        for (int e = threadIdx.x; e < nt * NCH; e += 128) {
-            const int r = e / NCH, c = e % NCH;
-            float dt = 0.0f, x = 0.0f;
-            if (ch0 + c < b.inner) { dt = softplus_(DT[(size_t)(row0 + n0 + r) * b.inner + ch0 + c]); x = XC[(size_t)(row0 + n0 + r) * b.inner + ch0 + c]; }
-            sdx[r][c] = make_float2(dt, dt * x);
-        }
-        __syncthreads();
-#pragma unroll 4
-        for (int r = 0; r < nt; r++) {
-            const float2 dx = sdx[r][ci];
-            float y = 0.0f;
+    __syncthreads();
+    auto row = [&](int buf, int r) {
+        const float2 dx = sdx[buf][r][ci];
+        float y = 0.0f;
 #pragma unroll
-            for (int k = 0; k < KS; k++) {
-                float a;
-                if (sizeof(OT) == 2) asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(a) : "f"(dx.x * A[k]));
-                else a = expf(dx.x * A[k]);
-                S[k] = fmaf(a, S[k], dx.y * sB[r][li * KS + k]);
-                y = fmaf(S[k], sC[r][li * KS + k], y);
-            }
+        for (int k = 0; k < KS; k++) {
+            float a;
+            if (sizeof(OT) == 2) asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(a) : "f"(dx.x * A[k]));
+            else a = expf(dx.x * A[k]);
+            S[k] = fmaf(a, S[k], dx.y * sB[buf][r][li * KS + k]);
+            y = fmaf(S[k], sC[buf][r][li * KS + k], y);
+        }
 #pragma unroll
-            for (int o = LANES / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-            if (li == 0) sy[r][ci] = y;
-        }
+        for (int o = LANES / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+        if (li == 0) sy[buf][r][ci] = y;
+    };
+    for (int it = 0; it < n_t; it++) {
+        const int nt = min(TILE, len - it * TILE), buf = it & 1;
+        if (nt == TILE) {
+#pragma unroll 8
+            for (int r = 0; r < TILE; r++) row(buf, r);
+        } else
+            for (int r = 0; r < nt; r++) row(buf, r);
         __syncthreads();
-        for (int e = threadIdx.x; e < nt * NCH; e += 128) {
-            const int r = e / NCH, c = e % NCH, cc = ch0 + c;
-            if (cc >= b.inner) continue;
-            const size_t row = row0 + n0 + r;
-            const float y = fmaf(b.D[cc], XC[row * b.inner + cc], sy[r][c]);
-            out[row * ld_out + b.a_off + cc] = cvt<OT>(y * silu_(P[row * ldp + b.z_off + cc]) * b.out_scale);
-        }
     }
     if (t.slots[slot].stopped) return;
 #pragma unroll
