@@ -796,7 +796,7 @@ struct SsmBranch {
 // XC [R][inner]: input behind its convolution; DT [R][inner]: step sizes before the softplus; BC [R][ld_bc]: columns dt_rank.. are B, then C.
 constexpr int SSM_SERVE = 384;
 template <typename OT, int LANES, int KS, int TILE>
-__global__ void __launch_bounds__(128 + SSM_SERVE) k_ssm_scan(PassTables t, SsmBranch b, const float* __restrict__ XC, const float* __restrict__ DT, const float* __restrict__ BC, int ld_bc,
+__global__ void __launch_bounds__(128 + SSM_SERVE, 1) k_ssm_scan(PassTables t, SsmBranch b, const float* __restrict__ XC, const float* __restrict__ DT, const float* __restrict__ BC, int ld_bc,
                                                   const float* __restrict__ P, int ldp, float* __restrict__ state, OT* __restrict__ out, int ld_out) {
     constexpr int NCH = 128 / LANES, NSP = LANES * KS, NE = (TILE * NCH + SSM_SERVE - 1) / SSM_SERVE;      // NE: (row, channel) pairs of a tile per serving thread
     __shared__ __align__(16) float sB[2][TILE][NSP], sC[2][TILE][NSP];
@@ -806,55 +806,72 @@ __global__ void __launch_bounds__(128 + SSM_SERVE) k_ssm_scan(PassTables t, SsmB
     const int slot = t.seg_slot[s], row0 = t.seg_row0[s], len = t.seg_len[s], n_t = (len + TILE - 1) / TILE;
     if (threadIdx.x >= 128) {
         const int tid = threadIdx.x - 128;
-        auto fill = [&](int it) {
-            const int n0 = it * TILE, nt = min(TILE, len - n0), buf = it & 1;
-            float x[NE], z[NE];
+        constexpr int NB = (TILE * NSP + SSM_SERVE - 1) / SSM_SERVE;
+        // what a tile needs waits in registers while the tile before it is served: no load is waited for
+        float fz[NE], fx[NE], fb[NB], fc[NB], dx[NE], dz[NE];
+        auto load_fill = [&](int it) {
+            const int n0 = it * TILE, nt = min(TILE, len - n0);       // (it >= n_t: nothing is on)
 #pragma unroll
             for (int i = 0; i < NE; i++) {
                 const int e = tid + i * SSM_SERVE, r = e / NCH, c = ch0 + e % NCH;
                 const bool on = r < nt && c < b.inner;
                 const size_t at = (size_t)(row0 + n0 + r) * b.inner + c;
-                z[i] = on ? DT[at] : 0.0f;
-                x[i] = on ? XC[at] : 0.0f;
+                fz[i] = on ? DT[at] : 0.0f;
+                fx[i] = on ? XC[at] : 0.0f;
             }
-            for (int e = tid; e < TILE * NSP; e += SSM_SERVE) {
-                const int r = e / NSP, n = e % NSP;
-                const float* p = BC + (size_t)(row0 + n0 + r) * ld_bc + b.dt_rank;
+#pragma unroll
+            for (int i = 0; i < NB; i++) {
+                const int e = tid + i * SSM_SERVE, r = e / NSP, n = e % NSP;
                 const bool on = r < nt && n < b.state;
-                sB[buf][r][n] = on ? p[n] : 0.0f;
-                sC[buf][r][n] = on ? p[b.state + n] : 0.0f;
+                const float* p = BC + (size_t)(row0 + n0 + r) * ld_bc + b.dt_rank + n;
+                fb[i] = on ? p[0] : 0.0f;
+                fc[i] = on ? p[b.state] : 0.0f;
+            }
+        };
+        auto put_fill = [&](int it) {
+            const int nt = min(TILE, len - it * TILE), buf = it & 1;
+#pragma unroll
+            for (int i = 0; i < NB; i++) {
+                const int e = tid + i * SSM_SERVE;
+                if (e < TILE * NSP) { sB[buf][e / NSP][e % NSP] = fb[i]; sC[buf][e / NSP][e % NSP] = fc[i]; }
             }
 #pragma unroll
             for (int i = 0; i < NE; i++) {
                 const int e = tid + i * SSM_SERVE;
-                const float dt = softplus_(z[i]);
-                if (e < TILE * NCH) sdx[buf][e / NCH][e % NCH] = make_float2(dt, dt * x[i]);
+                const float dt = e / NCH < nt ? softplus_(fz[i]) : 0.0f;      // rows behind the segment leave the state as it is
+                if (e < TILE * NCH) sdx[buf][e / NCH][e % NCH] = make_float2(dt, dt * fx[i]);
             }
         };
-        auto drain = [&](int it) {
-            const int n0 = it * TILE, nt = min(TILE, len - n0), buf = it & 1;
-            float x[NE], z[NE];
+        auto load_drain = [&](int it) {
+            const int n0 = it * TILE, nt = min(TILE, len - n0);
 #pragma unroll
             for (int i = 0; i < NE; i++) {
                 const int e = tid + i * SSM_SERVE, r = e / NCH, c = ch0 + e % NCH;
                 const bool on = r < nt && c < b.inner;
-                x[i] = on ? b.D[c] * XC[(size_t)(row0 + n0 + r) * b.inner + c] : 0.0f;
-                z[i] = on ? P[(size_t)(row0 + n0 + r) * ldp + b.z_off + c] : 0.0f;
+                dx[i] = on ? b.D[c] * XC[(size_t)(row0 + n0 + r) * b.inner + c] : 0.0f;
+                dz[i] = on ? P[(size_t)(row0 + n0 + r) * ldp + b.z_off + c] : 0.0f;
             }
+        };
+        auto put_drain = [&](int it) {
+            const int n0 = it * TILE, nt = min(TILE, len - n0), buf = it & 1;
 #pragma unroll
             for (int i = 0; i < NE; i++) {
                 const int e = tid + i * SSM_SERVE, r = e / NCH, c = ch0 + e % NCH;
-                if (r < nt && c < b.inner) out[(size_t)(row0 + n0 + r) * ld_out + b.a_off + c] = cvt<OT>((sy[buf][r][e % NCH] + x[i]) * (sizeof(OT) == 2 ? __fdividef(z[i], 1.0f + __expf(-z[i])) : silu_(z[i])) * b.out_scale);
+                if (r < nt && c < b.inner)
+                    out[(size_t)(row0 + n0 + r) * ld_out + b.a_off + c] = cvt<OT>((sy[buf][r][e % NCH] + dx[i]) * (sizeof(OT) == 2 ? __fdividef(dz[i], 1.0f + __expf(-dz[i])) : silu_(dz[i])) * b.out_scale);
             }
         };
-        fill(0);
+        load_fill(0);
+        put_fill(0);
+        load_fill(1);
         __syncthreads();
         for (int it = 0; it < n_t; it++) {
-            if (it + 1 < n_t) fill(it + 1);
-            if (it > 0) drain(it - 1);
+            if (it + 1 < n_t) { put_fill(it + 1); load_fill(it + 2); }
+            if (it > 0) put_drain(it - 1);
+            load_drain(it);
             __syncthreads();
         }
-        drain(n_t - 1);
+        put_drain(n_t - 1);
         return;
     }
     const int ci = threadIdx.x / LANES, li = threadIdx.x % LANES, ch = ch0 + ci;
@@ -870,28 +887,56 @@ __global__ void __launch_bounds__(128 + SSM_SERVE) k_ssm_scan(PassTables t, SsmB
         if (sizeof(OT) == 2) A[k] *= 1.4426950408889634f;
     }
     __syncthreads();
-    auto row = [&](int buf, int r) {
-        const float2 dx = sdx[buf][r][ci];
-        float y = 0.0f;
-#pragma unroll
-        for (int k = 0; k < KS; k++) {
-            float a;
-            if (sizeof(OT) == 2) asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(a) : "f"(dx.x * A[k]));
-            else a = expf(dx.x * A[k]);
-            S[k] = fmaf(a, S[k], dx.y * sB[buf][r][li * KS + k]);
-            y = fmaf(S[k], sC[buf][r][li * KS + k], y);
-        }
-#pragma unroll
-        for (int o = LANES / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-        if (li == 0) sy[buf][r][ci] = y;
-    };
+    // NR rows at a time: their loads and decays are independent of the state, and their read-outs are summed over the channel's lanes together (a lane
+    // ends with NR / LANES of them)
+    constexpr int NR = KS == 4 ? 8 : 4;
     for (int it = 0; it < n_t; it++) {
         const int nt = min(TILE, len - it * TILE), buf = it & 1;
-        if (nt == TILE) {
-#pragma unroll 8
-            for (int r = 0; r < TILE; r++) row(buf, r);
-        } else
-            for (int r = 0; r < nt; r++) row(buf, r);
+        for (int r0 = 0; r0 < nt; r0 += NR) {
+            float a[NR][KS], w[NR][KS], c[NR][KS], y[NR];
+#pragma unroll
+            for (int j = 0; j < NR; j++) {
+                const float2 dx = sdx[buf][r0 + j][ci];
+#pragma unroll
+                for (int k = 0; k < KS; k += 4) {
+                    const float4 b4 = *reinterpret_cast<const float4*>(&sB[buf][r0 + j][li * KS + k]), c4 = *reinterpret_cast<const float4*>(&sC[buf][r0 + j][li * KS + k]);
+                    w[j][k] = dx.y * b4.x; w[j][k + 1] = dx.y * b4.y; w[j][k + 2] = dx.y * b4.z; w[j][k + 3] = dx.y * b4.w;
+                    c[j][k] = c4.x; c[j][k + 1] = c4.y; c[j][k + 2] = c4.z; c[j][k + 3] = c4.w;
+                }
+#pragma unroll
+                for (int k = 0; k < KS; k++) {
+                    if (sizeof(OT) == 2) asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(a[j][k]) : "f"(dx.x * A[k]));
+                    else a[j][k] = expf(dx.x * A[k]);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < NR; j++) {
+                y[j] = 0.0f;
+#pragma unroll
+                for (int k = 0; k < KS; k++) { S[k] = fmaf(a[j][k], S[k], w[j][k]); y[j] = fmaf(S[k], c[j][k], y[j]); }
+            }
+            int rb = r0;
+            bool first = true;                            // among the lanes that end with the same rows
+#pragma unroll
+            for (int o = LANES / 2, n = NR; o > 0; o >>= 1, n = n > 1 ? n / 2 : 1) {
+                if (n > 1) {
+                    const bool up = (li & o) != 0;
+#pragma unroll
+                    for (int j = 0; j < NR / 2; j++) {
+                        if (j >= n / 2) continue;
+                        const float give = up ? y[j] : y[j + n / 2], keep = up ? y[j + n / 2] : y[j];
+                        y[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+                    }
+                    rb += up ? n / 2 : 0;
+                } else {
+                    y[0] += __shfl_xor_sync(0xffffffffu, y[0], o);
+                    first = first && (li & o) == 0;
+                }
+            }
+            constexpr int LEFT = NR > LANES ? NR / LANES : 1;
+#pragma unroll
+            for (int j = 0; j < LEFT; j++) if (first) sy[buf][rb + j][ci] = y[j];
+        }
         __syncthreads();
     }
     if (t.slots[slot].stopped) return;
