@@ -84,17 +84,17 @@ enum { GTB_ROT_SCALE_WAVES = 0, GTB_ROT_SCALE_YARN = 1 };         /* how rot_fac
  *    sink 2: the sink's score is 0 for every head (no tensor): the denominator holds one more 1.  out_bias: the out projection adds the
  *    vector o.b (single-branch layers, both attention kinds).
  *  Recurrent mixers of sandwich layers (fp32 state per slot, gates, decays, step sizes and unit norms in fp32):
- *  GTB_MIX_MLSTM: per head log gates i = gate_cap tanh((i h + i.b) / gate_cap), f = log logistic(gate_cap tanh((f h + f.b) / gate_cap)); with
- *    m_0 = 0, m_t = max(f + m_(t-1), i): S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k v^T, the vector n_t likewise with k alone, both from
- *    zero; o = S_t^T q / (max(|n_t . q|, exp(-m_t)) + 1e-6), q scaled by `scale`; per head o to unit RMS (eps of the model), times `norm`
- *    [heads * vdim], times logistic(g h).  Tensors q, k, v, g, i, i.b, f, f.b, norm, o.
+ *  GTB_MIX_MLSTM: cap(z) = gate_cap tanh(z / gate_cap); per head a log input gate a = cap(i h + i.b) and a log decay d = log logistic(cap(f h + f.b)).
+ *    A running maximum r, 0 in an empty slot, becomes r' = max(d + r, a); the memory becomes e^(d + r - r') M + e^(a - r') k v^T and its normaliser
+ *    e^(d + r - r') c + e^(a - r') k (M and c empty at first).  Read-out M^T q / (max(|c . q|, e^-r') + 1e-6) with q times `scale`, per head to unit RMS
+ *    (eps of the model), times `norm` [heads * vdim], times logistic(g h).  Tensors q, k, v, g, i, i.b, f, f.b, norm, o.
  *  GTB_MIX_DELTA: q, k (kv_heads heads; head h uses h / (heads / kv_heads)) and v each pass a causal convolution of `conv` taps per channel (as
- *    below, no bias) and silu; q and k divided by sqrt(sum of squares + 1e-6), q times `scale`; g_t = exp(-exp(A_log) softplus(a h + dt_bias)),
- *    beta = logistic(b h) per head; S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q; per head o to unit RMS times `norm` [vdim], times
- *    silu(g h).  Tensors q, k, v, q.conv, k.conv, v.conv, g, b, a, A_log, dt_bias, norm, o.
+ *    below, no bias) and silu; q and k divided by sqrt(sum of squares + 1e-6), q times `scale`; per head a decay e^(-exp(A_log) softplus(a h +
+ *    dt_bias)) and a rate w = logistic(b h).  The memory M first decays, then moves by w k (v - M^T k)^T, then is read: M^T q, per head to unit RMS times
+ *    `norm` [vdim], times silu(g h).  Tensors q, k, v, q.conv, k.conv, v.conv, g, b, a, A_log, dt_bias, norm, o.
  *  GTB_MIX_SSM: selective scan over `inner` channels with `state` numbers each: [x | z] = in h; x passes the convolution of `conv` taps with bias
- *    conv.b and silu; [d | B | C] = x_proj x (dt_rank, state, state rows of tensor x), dt = softplus(dt d + dt.b), S[c][n] <- exp(-dt_c
- *    exp(A_log[c][n])) S[c][n] + dt_c x_c B_n, y_c = sum_n S[c][n] C_n + D_c x_c; output o (y * silu(z)).  Tensors in, conv, conv.b, x, dt,
+ *    conv.b and silu; [d | B | C] = x_proj x (dt_rank, state, state rows of tensor x), step s = softplus(dt d + dt.b); the numbers of
+ *    channel c decay by e^(-s_c exp(A_log)) and gain s_c x_c B; the channel's value is their product with C plus D_c x_c; output o (value * silu(z)).  Tensors in, conv, conv.b, x, dt,
  *    dt.b, A_log, D, o.
  *    retention -- act 1: q, k, v <- silu(q), silu(k), silu(v) before the recurrence; out_norm 2: the concatenated heads are scaled to
  *    unit RMS TOGETHER and multiplied by the weight `norm` [heads * vdim]; gated 2: times logistic(g h). */

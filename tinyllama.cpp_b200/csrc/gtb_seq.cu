@@ -20,6 +20,8 @@
 //    kernels of the other styles (softmax attention, retention) side by side, each weighted by out_scale in the out-projection operand --
 //    or latent attention alone.  Queries and keys that pass a convolution behind their projections leave the raw projection in place (its
 //    last rows become the slot's history): the queries go to a buffer of their own, the keys to the cache.
+//    Recurrent mixers (mLSTM, delta rule, selective scan) run from the projections or from their convolved copy; joined branches have an out projection
+//    each, on k-block borders of the one out matrix.  A layer that is an earlier one once more has no LayerW content: its run names the other layer.
 //    Group-limited experts reuse the stacked layout of the post-norm experts; the shared expert is cut along its inner width into parts of
 //    one expert's size that follow the routed experts in the same stacks, so every row simply has `top + parts` choices.
 #include <math.h>

@@ -1,8 +1,8 @@
 // gtb_seq_recur.cuh -- recurrent token mixers whose decay depends on the token, for the layer-list sequence models:
 //   * "mLSTM": S <- a_t S + w_t k_t [v_t | 1]^T per head, a and w from a capped exponential input gate and a logistic forget gate under a
 //     running maximum; the column of ones is the normaliser, so it needs no kernel of its own
-//   * gated delta rule: S <- g_t S; u = beta_t (v_t - S^T k_t); S <- S + k_t u^T; unit-length q and k
-//   * selective scan (Mamba): S[c][n] <- exp(dt_c A[c][n]) S[c][n] + dt_c x_c B_n, y_c = sum_n S[c][n] C_n + D_c x_c
+//   * gated delta rule: S decays by g_t, then moves by beta_t k_t (v_t - S^T k_t)^T, then is read with q_t; unit-length q and k
+//   * selective scan (Mamba): every channel holds a row of numbers that decay by e^(step A) and gain step x B, read out with C
 // Rows are walked one by one from the slot's state (decode rows, short portions, float mode); prompt portions in bf16 mode take the first two
 // chunk-wise on tensor cores.
 //
@@ -43,10 +43,6 @@ __device__ __forceinline__ float softplus_series(float z) {
     p = fmaf(q, p, 1.0f);
     return fmaxf(z, 0.0f) + 2.0f * s * p;
 }
-__device__ __forceinline__ void split2(float v, bf16& hi, bf16& lo) {
-    hi = __float2bfloat16_rn(v);
-    lo = __float2bfloat16_rn(v - __bfloat162float(hi));
-}
 // two neighbouring values as packed hi and lo pairs
 __device__ __forceinline__ void split2_pack(float a, float b, uint32_t& hi, uint32_t& lo) {
     hi = sa_pack(a, b);
@@ -54,8 +50,8 @@ __device__ __forceinline__ void split2_pack(float a, float b, uint32_t& hi, uint
 }
 
 // ------------------------------------------------------------------------------------------------ gates
-// log decay la and input weight w of one (row, head).  mLSTM: i = cap tanh(z_i / cap), f = log logistic(cap tanh(z_f / cap));
-// delta rule: la = -exp(A_log) softplus(z + dt_bias), w = logistic(z_b)
+// log decay la and input weight w of one (row, head).  mLSTM: capped log input gate i and log forget gate f (their combination needs the
+// running maximum); delta rule: la from the step size softplus(z + dt_bias), w = logistic
 __device__ __forceinline__ void mlstm_gates(const RecBranch& b, const float* __restrict__ p, int h, float& i, float& f) {
     i = b.cap * tanhf(p[b.i_off + h] / b.cap);
     f = -softplus_(-b.cap * tanhf(p[b.f_off + h] / b.cap));
@@ -64,8 +60,8 @@ __device__ __forceinline__ void delta_gates(const RecBranch& b, const float* __r
     la = -expf(b.A_log[h]) * softplus_(p[b.i_off + h] + b.dt_bias[h]);
     w = sigmoidf_(p[b.f_off + h]);
 }
-// G [R][heads]: {log decay, w, m, 0}.  mLSTM: with m_t = max(f + m_(t-1), i) the row's decay is exp(f + m_(t-1) - m_t) and its input weight
-// exp(i - m_t) times the query scale (w holds the logarithm; every factor is at most 1); delta rule: w = beta.
+// G [R][heads]: {log decay, w, m, 0}.  mLSTM: the running maximum goes from m' to m = max(f + m', i); the row's decay is e^(f + m' - m) and its
+// input weight e^(i - m) times the query scale (w holds the logarithm; every factor is at most 1); delta rule: w = beta.
 // Bp [R][heads] (or null): the sum of the log decays from the start of the row's chunk of C rows, as hi + lo (summed in double), so that
 // differences of two sums keep their precision.  The running maximum is a max-plus scan: rows compose as (F, M) o (F', M') =
 // (F + F', max(M + F', M')).  grid (segments, heads); blockDim a multiple of C (or 32 without Bp).
